@@ -1173,16 +1173,17 @@ DSB_EXPORT int dsb200_paged_flash_window(const void* q, long long q_tok_stride, 
 // bf16 at q_tok_stride elements per token (a multiple of 8), kv_cache [num_blocks][2][block_size][hkv][head_dim] bf16; out rows at out_ld
 // elements per token (a multiple of 8).  decode != 0 selects the small-atom kernel (head_dim 128, q:kv head ratios dividing 16).
 // sink_logit (hq floats): learned sinks, exp(sink_logit[h]) joins head h's denominator; r1, r2 (hq floats each): the score of key j for the
-// query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions.  Each may
-// be absent (null / 0).
+// query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions;
+// window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0).
 DSB_EXPORT int dsb200_paged_flash_sink_ex(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld, const int* tok_seq,
                                        const int* tok_pos, const int* block_table, int n_tokens, int hq, int hkv, int head_dim, int block_size,
                                        int max_blocks_per_seq, int num_blocks, float scale, float softcap, float sink, const float* sink_logit,
-                                       const float* r1, const float* r2, int part, int max_atoms, int n_splits, void* scratch, int decode,
+                                       const float* r1, const float* r2, int part, int window, int max_atoms, int n_splits, void* scratch, int decode,
                                        cudaStream_t stream) {
   using namespace dsb;
   if (n_tokens == 0) return DSB_OK;
-  DSB_REQUIRE((r1 == nullptr) == (r2 == nullptr) && part >= 0 && (r1 == nullptr || softcap == 0.f), "paged_flash_sink: distance term / part %d", part);
+  DSB_REQUIRE((r1 == nullptr) == (r2 == nullptr) && part >= 0 && window >= 0 && (part == 0 || window == 0) && (r1 == nullptr || softcap == 0.f),
+              "paged_flash_sink: distance term / part %d / window %d", part, window);
   paged::MaskExtras ex;
   ex.sink_logit = sink_logit; ex.r1 = r1; ex.r2 = r2; ex.part = part;
   DSB_REQUIRE(head_dim == 64 || head_dim == 128, "paged_flash_sink: head_dim %d unsupported (64 or 128)", head_dim);
@@ -1194,13 +1195,13 @@ DSB_EXPORT int dsb200_paged_flash_sink_ex(const void* q, long long q_tok_stride,
   if (decode) {
     DSB_REQUIRE(head_dim == 128 && 16 % (hq / hkv) == 0, "paged_flash_sink: the decode kernel takes head_dim 128 and head ratios dividing 16");
     return paged::launch_decode(q, kv_cache, out, tok_seq, tok_pos, block_table, n_tokens, hq, hkv, block_size, max_blocks_per_seq, num_blocks, scale,
-                                max_atoms, n_splits, scratch, nullptr, 0, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
+                                max_atoms, n_splits, scratch, nullptr, window, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
   }
   if (head_dim == 128)
     return paged::launch<128>(q, kv_cache, out, tok_seq, tok_pos, block_table, n_tokens, hq, hkv, block_size, max_blocks_per_seq, num_blocks, scale,
-                              max_atoms, n_splits, scratch, nullptr, 0, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
+                              max_atoms, n_splits, scratch, nullptr, window, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
   return paged::launch<64>(q, kv_cache, out, tok_seq, tok_pos, block_table, n_tokens, hq, hkv, block_size, max_blocks_per_seq, num_blocks, scale,
-                           max_atoms, n_splits, scratch, nullptr, 0, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
+                           max_atoms, n_splits, scratch, nullptr, window, stream, hq, head_dim, q_tok_stride, 2, 0, out_ld, 1.f, softcap, sink, ex);
 }
 
 DSB_EXPORT int dsb200_paged_flash_sink(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld, const int* tok_seq,
@@ -1208,6 +1209,6 @@ DSB_EXPORT int dsb200_paged_flash_sink(const void* q, long long q_tok_stride, co
                                        int max_blocks_per_seq, int num_blocks, float scale, float softcap, float sink, int max_atoms, int n_splits,
                                        void* scratch, int decode, cudaStream_t stream) {
   return dsb200_paged_flash_sink_ex(q, q_tok_stride, kv_cache, out, out_ld, tok_seq, tok_pos, block_table, n_tokens, hq, hkv, head_dim, block_size,
-                                    max_blocks_per_seq, num_blocks, scale, softcap, sink, nullptr, nullptr, nullptr, 0, max_atoms, n_splits, scratch,
+                                    max_blocks_per_seq, num_blocks, scale, softcap, sink, nullptr, nullptr, nullptr, 0, 0, max_atoms, n_splits, scratch,
                                     decode, stream);
 }

@@ -7,6 +7,7 @@
 //   embed_sinusoid        token table lookup + sinusoidal position vector -> fp32 residual
 //   sandwich_norm         x += rms(y) * (wb + ob)   and / or   out = rms(x) * (w + o)      (one pass per token row)
 //   stream_group_norm     x += y0 + y1 + y2         and / or   out = rms-in-groups(x) * w      (blocks whose sublayers share one norm)
+//   stream_tanh_norm      x += y0 + y1 + y2         and / or   out = tanh(alpha x) * w + b           (the same with a norm that has no statistic)
 //   latent_norm_append    plain-weight RMS norm of the query latent and of the key/value latent of every token; the
 //                         key/value latent goes straight into its slot of the paged latent cache
 //   latent_attention      softmax(q_abs . c) c over the paged latent cache: all heads of a token share the cached rows
@@ -320,6 +321,48 @@ __global__ void stream_group_norm_vec_kernel(float* __restrict__ x, const TY* __
 
 // One warp per (token, which): which = 0 normalises lat[t, :nq] with wq into cq[t, :]; which = 1 normalises
 // lat[t, nq : nq + nkv] with wkv into the token's row of the paged cache [blocks, block_size, nkv].
+// The same block with a "norm" that looks at no other value of the row: out = tanh(alpha x) * w + b after the finished outputs have joined the
+// stream.  There is nothing to reduce, so a thread owns V consecutive values (V = 4: dim and every base a multiple of 16 bytes) of any row.
+template <typename TY, typename TO, int V>
+__global__ void __launch_bounds__(256)
+stream_tanh_norm_kernel(float* __restrict__ x, const TY* __restrict__ y0, const TY* __restrict__ y1, const float* __restrict__ y2,
+                        const float* __restrict__ alpha, const float* __restrict__ w, const float* __restrict__ b, TO* __restrict__ out,
+                        float* __restrict__ out32, const int* __restrict__ rows, long long n, int dim) {
+  const float al = w ? *alpha : 0.f;
+  const int per = dim / V;
+  const bool add = y0 != nullptr || y1 != nullptr || y2 != nullptr;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / per;
+    const int c = static_cast<int>(i - r * per) * V;
+    const size_t so = static_cast<size_t>(rows ? rows[r] : r) * dim + c, o = static_cast<size_t>(r) * dim + c;
+    if constexpr (V == 4) {
+      float4 v = load4(x + so);
+      if (y0) { const float4 a = load4(y0 + so); v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+      if (y1) { const float4 a = load4(y1 + so); v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+      if (y2) { const float4 a = load4(y2 + so); v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+      if (add && rows == nullptr) store4(x + so, v);
+      if (w != nullptr) {
+        const float4 g = load4(w + c), s = load4(b + c);
+        const float4 t = make_float4(fmaf(tanhf(al * v.x), g.x, s.x), fmaf(tanhf(al * v.y), g.y, s.y), fmaf(tanhf(al * v.z), g.z, s.z),
+                                     fmaf(tanhf(al * v.w), g.w, s.w));
+        store4(out + o, t);
+        if (out32) store4(out32 + o, t);
+      }
+    } else {
+      float v = x[so];
+      if (y0) v += to_f(y0[so]);
+      if (y1) v += to_f(y1[so]);
+      if (y2) v += y2[so];
+      if (add && rows == nullptr) x[so] = v;
+      if (w != nullptr) {
+        const float t = fmaf(tanhf(al * v), w[c], b[c]);
+        out[o] = from_f<TO>(t);
+        if (out32) out32[o] = t;
+      }
+    }
+  }
+}
+
 template <typename T>
 __global__ void latent_norm_append_kernel(const T* __restrict__ lat, int ld, const float* __restrict__ wq, const float* __restrict__ wkv,
                                           T* __restrict__ cq, T* __restrict__ cache, const int* __restrict__ tok_seq,
@@ -567,9 +610,10 @@ __global__ void clamped_swish_gate_vec_kernel(const T* __restrict__ gu, T* __res
   }
 }
 
-// The same on column ranges: gate at column gate_col0 and up at column up_col0 of gu [rows, ld], result into out [rows, out_ld] (a view)
+// The same on column ranges: gate at column gate_col0 and up at column up_col0 of gu [rows, ld], result into out [rows, out_ld] (a view).
+// row_col >= 0: the whole row is multiplied by the sigmoid of the number in that column of gu (one gate per token).
 template <typename T>
-__global__ void clamped_swish_gate_cols_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, T* __restrict__ out,
+__global__ void clamped_swish_gate_cols_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, int row_col, T* __restrict__ out,
                                                long long out_ld, long long rows, int F, float alpha, float limit, float shift) {
   const long long n = rows * F;
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
@@ -577,13 +621,14 @@ __global__ void clamped_swish_gate_cols_kernel(const T* __restrict__ gu, long lo
     const int c = static_cast<int>(i % F);
     const float g = fminf(to_f(gu[r * ld + gate_col0 + c]), limit);
     const float u = fminf(fmaxf(to_f(gu[r * ld + up_col0 + c]), -limit), limit);
-    out[r * out_ld + c] = from_f<T>(g * (1.f / (1.f + expf(-alpha * g))) * (u + shift));
+    const float rg = row_col >= 0 ? 1.f / (1.f + expf(-to_f(gu[r * ld + row_col]))) : 1.f;
+    out[r * out_ld + c] = from_f<T>(g * (1.f / (1.f + expf(-alpha * g))) * (u + shift) * rg);
   }
 }
 
 // ... with F, both column offsets and both row strides multiples of 4 and 16-byte (fp32) / 8-byte (bf16) aligned bases: four outputs per thread
 template <typename T>
-__global__ void clamped_swish_gate_cols_vec_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, T* __restrict__ out,
+__global__ void clamped_swish_gate_cols_vec_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, int row_col, T* __restrict__ out,
                                                    long long out_ld, long long rows, int F, float alpha, float limit, float shift) {
   const int fv = F >> 2;
   const long long n = rows * fv;
@@ -592,12 +637,13 @@ __global__ void clamped_swish_gate_cols_vec_kernel(const T* __restrict__ gu, lon
     const int c = static_cast<int>(i % fv) * 4;
     const float4 g4 = load4(gu + r * ld + gate_col0 + c), u4 = load4(gu + r * ld + up_col0 + c);
     const float gs[4] = {g4.x, g4.y, g4.z, g4.w}, us[4] = {u4.x, u4.y, u4.z, u4.w};
+    const float rg = row_col >= 0 ? 1.f / (1.f + expf(-to_f(gu[r * ld + row_col]))) : 1.f;
     float o[4];
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
       const float g = fminf(gs[k], limit);
       const float u = fminf(fmaxf(us[k], -limit), limit);
-      o[k] = g * (1.f / (1.f + expf(-alpha * g))) * (u + shift);
+      o[k] = g * (1.f / (1.f + expf(-alpha * g))) * (u + shift) * rg;
     }
     store4(out + r * out_ld + c, make_float4(o[0], o[1], o[2], o[3]));
   }
@@ -612,7 +658,7 @@ __global__ void softcap_kernel(float* __restrict__ x, long long ld, int cols, lo
 
 // ---------------------------------------------------------------------------------------------------------------------- router
 // One warp per token.  Shared memory per warp: E selection scores + G group scores.  Ties go to the lower index.
-__global__ void grouped_topk_gating_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ expert_counts,
+__global__ void grouped_topk_gating_kernel(const float* __restrict__ logits, const float* __restrict__ bias, const float* __restrict__ correction, int* __restrict__ expert_counts,
                                            float* __restrict__ scores, int* __restrict__ assignments, int* __restrict__ offsets, int n_tokens,
                                            int E, int K, int G, int keep, int normalize, int sigmoid_scores) {
   extern __shared__ float smem[];
@@ -621,20 +667,21 @@ __global__ void grouped_topk_gating_kernel(const float* __restrict__ logits, con
   if (tok >= n_tokens) return;
   float* choice = smem + static_cast<size_t>(wib) * (E + G);
   float* gsc = choice + E;
-  const float* lg = logits + static_cast<size_t>(tok) * E;
+  const float* row = logits + static_cast<size_t>(tok) * E;
+  auto lg = [&](int e) { return bias ? row[e] + bias[e] : row[e]; };
   float mx = 0.f, inv = 1.f;
   if (!sigmoid_scores) {
     mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg[e]);
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, lg(e));
     mx = warp_max(mx);
     float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(lg[e] - mx);
+    for (int e = lane; e < E; e += 32) sum += expf(lg(e) - mx);
     sum = warp_sum(sum);
     inv = 1.f / sum;
   }
   // score of expert e: its softmax probability, or (sigmoid_scores) 1 / (1 + exp(-logit)) on its own
   for (int e = lane; e < E; e += 32)
-    choice[e] = (sigmoid_scores ? 1.f / (1.f + expf(-lg[e])) : expf(lg[e] - mx) * inv) + (correction ? correction[e] : 0.f);
+    choice[e] = (sigmoid_scores ? 1.f / (1.f + expf(-lg(e))) : expf(lg(e) - mx) * inv) + (correction ? correction[e] : 0.f);
   __syncwarp();
   if (G > 1 && keep < G) {
     const int per = E / G;
@@ -674,7 +721,7 @@ __global__ void grouped_topk_gating_kernel(const float* __restrict__ logits, con
     }
     float s = 0.f;
     if (best_e >= 0) {
-      s = sigmoid_scores ? 1.f / (1.f + expf(-lg[best_e])) : expf(lg[best_e] - mx) * inv;
+      s = sigmoid_scores ? 1.f / (1.f + expf(-lg(best_e))) : expf(lg(best_e) - mx) * inv;
       if (lane == 0) choice[best_e] = -INFINITY;
     }
     __syncwarp();
@@ -915,6 +962,32 @@ DSB_EXPORT int dsb200_stream_group_norm(float* x, const void* y0, const void* y1
   return DSB_OK;
 }
 
+// `dsb200_stream_group_norm` with out[r] = tanh(alpha * row) * w + b in place of the RMS norm: alpha one float on the device, w and b [dim].
+DSB_EXPORT int dsb200_stream_tanh_norm(float* x, const void* y0, const void* y1, int y_dtype, const float* y2, const float* alpha, const float* w,
+                                       const float* b, void* out, int out_dtype, float* out32, const int* rows, int n_rows, int dim,
+                                       cudaStream_t stream) {
+  if (n_rows == 0) return DSB_OK;
+  DSB_REQUIRE(w == nullptr || (out != nullptr && alpha != nullptr && b != nullptr), "stream_tanh_norm: a norm needs alpha, a shift and an output");
+  const uintptr_t all = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y0) | reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(y2) |
+                        reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(out32);
+  const bool vec = dim % 4 == 0 && (all & 15) == 0;
+  const long long n = static_cast<long long>(n_rows) * (vec ? dim / 4 : dim);
+#define LAUNCH(TY, TO)                                                                                                                              \
+  do {                                                                                                                                              \
+    if (vec)                                                                                                                                        \
+      stream_tanh_norm_kernel<TY, TO, 4><<<grid_for(n, 256), 256, 0, stream>>>(x, (const TY*)y0, (const TY*)y1, y2, alpha, w, b, (TO*)out, out32, rows, n, dim); \
+    else                                                                                                                                            \
+      stream_tanh_norm_kernel<TY, TO, 1><<<grid_for(n, 256), 256, 0, stream>>>(x, (const TY*)y0, (const TY*)y1, y2, alpha, w, b, (TO*)out, out32, rows, n, dim); \
+  } while (0)
+  if (y_dtype == 0 && out_dtype == 0) LAUNCH(bf16, bf16);
+  else if (y_dtype == 0) LAUNCH(bf16, float);
+  else if (out_dtype == 0) LAUNCH(float, bf16);
+  else LAUNCH(float, float);
+#undef LAUNCH
+  DSB_CHECK_CUDA(cudaGetLastError());
+  return DSB_OK;
+}
+
 // lat [n_tokens, ld] holds (query latent [nq] | key/value latent [nkv]) of every token.  cq [n_tokens, nq] = plain-weight RMS norm
 // of the first part; the RMS-normed second part is written to the token's row of cache [blocks, block_size, cache_ld] (cache_ld >= nkv:
 // rows may be padded to a width the tensor-core attention takes; the padding is never written).
@@ -1038,24 +1111,25 @@ DSB_EXPORT int dsb200_clamped_swish_gate(const void* gu, void* out, long long ro
 
 // out[r, c] = g' * sigmoid(alpha g') * (clamp(u, -limit, limit) + shift) with g' = min(gu[r, gate_col0 + c], limit), u = gu[r, up_col0 + c], c < F:
 // gate and up are column ranges of one fused projection gu [rows, ld]; out [rows, out_ld] may be a column range of a wider buffer.
-DSB_EXPORT int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, void* out, long long out_ld, long long rows,
-                                              int F, float alpha, float limit, float shift, int dtype, cudaStream_t stream) {
+// row_col >= 0: row r is also multiplied by sigmoid(gu[r, row_col]).
+DSB_EXPORT int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, int row_col, void* out, long long out_ld,
+                                              long long rows, int F, float alpha, float limit, float shift, int dtype, cudaStream_t stream) {
   const long long n = rows * F;
   if (n == 0) return DSB_OK;
   const int esz = dtype == 0 ? 2 : 4;
   const bool vec = F % 4 == 0 && gate_col0 % 4 == 0 && up_col0 % 4 == 0 && ld % 4 == 0 && out_ld % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & (4 * esz - 1)) == 0;
   if (vec && dtype == 0)
-    clamped_swish_gate_cols_vec_kernel<bf16><<<grid_for(n / 4, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, (bf16*)out, out_ld, rows, F,
+    clamped_swish_gate_cols_vec_kernel<bf16><<<grid_for(n / 4, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, row_col, (bf16*)out, out_ld, rows, F,
                                                                                      alpha, limit, shift);
   else if (vec)
-    clamped_swish_gate_cols_vec_kernel<float><<<grid_for(n / 4, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, (float*)out, out_ld, rows, F,
+    clamped_swish_gate_cols_vec_kernel<float><<<grid_for(n / 4, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, row_col, (float*)out, out_ld, rows, F,
                                                                                       alpha, limit, shift);
   else if (dtype == 0)
-    clamped_swish_gate_cols_kernel<bf16><<<grid_for(n, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, (bf16*)out, out_ld, rows, F, alpha,
+    clamped_swish_gate_cols_kernel<bf16><<<grid_for(n, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, row_col, (bf16*)out, out_ld, rows, F, alpha,
                                                                               limit, shift);
   else
-    clamped_swish_gate_cols_kernel<float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, (float*)out, out_ld, rows, F,
+    clamped_swish_gate_cols_kernel<float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, row_col, (float*)out, out_ld, rows, F,
                                                                                alpha, limit, shift);
   DSB_CHECK_CUDA(cudaGetLastError());
   return DSB_OK;
@@ -1070,12 +1144,13 @@ DSB_EXPORT int dsb200_softcap(float* x, long long ld, long long rows, int cols, 
   return DSB_OK;
 }
 
-// Router: scores = softmax over the E logits of a token, or (sigmoid_scores) the sigmoid of every logit on its own; selection score =
+// Router: scores = softmax over the E logits of a token (bias[e], when given, joins the logits first), or (sigmoid_scores) the sigmoid of every
+// logit on its own; selection score =
 // score + correction[e] (correction may be null); experts are split
 // into `groups` contiguous groups of equal size, of which the `keep` with the largest maximal selection score stay selectable; the top_k
 // selectable experts by selection score are assigned; their weights are the uncorrected scores (divided by their sum when
 // `normalize`).  Outputs as dsb200_top_k_gating; expert_counts must be zeroed by the caller.
-DSB_EXPORT int dsb200_grouped_topk_gating(const float* logits, const float* correction, int* expert_counts, float* scores, int* assignments,
+DSB_EXPORT int dsb200_grouped_topk_gating(const float* logits, const float* bias, const float* correction, int* expert_counts, float* scores, int* assignments,
                                           int* offsets, int n_tokens, int n_experts, int top_k, int groups, int keep, int normalize,
                                           int sigmoid_scores, cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
@@ -1085,7 +1160,7 @@ DSB_EXPORT int dsb200_grouped_topk_gating(const float* logits, const float* corr
               "grouped_topk_gating: %d experts in %d groups, %d kept, top %d", n_experts, groups, keep, top_k);
   const int wpb = 4;
   const size_t smem = static_cast<size_t>(wpb) * (n_experts + groups) * sizeof(float);
-  grouped_topk_gating_kernel<<<(n_tokens + wpb - 1) / wpb, wpb * 32, smem, stream>>>(logits, correction, expert_counts, scores, assignments,
+  grouped_topk_gating_kernel<<<(n_tokens + wpb - 1) / wpb, wpb * 32, smem, stream>>>(logits, bias, correction, expert_counts, scores, assignments,
                                                                                    offsets, n_tokens, n_experts, top_k, groups, keep, normalize, sigmoid_scores);
   DSB_CHECK_CUDA(cudaGetLastError());
   return DSB_OK;

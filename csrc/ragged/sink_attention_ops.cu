@@ -5,6 +5,8 @@
 //                             shared by the heads, then the first rot_dims entries of the head are rotated (entry i paired with entry
 //                             i + rot_dims / 2) by pos * freq[i], cosine and sine times a constant; every value head is divided by its own
 //                             root mean square (no weight).  Queries leave as a tensor, keys and values go to their rows of the paged cache.
+//                             Norms, biases (added first) and the key / value part are optional: a layer that reads another layer's cache
+//                             only prepares its queries.
 //   sink_attention            causal attention over the paged cache on CUDA cores: score = scale q . k, optionally soft-capped
 //                             (cap tanh(score / cap)); weights exp(s_j) / (sink + sum_j exp(s_j)) with sink = 1 for a softmax that has
 //                             one more, valueless entry of score 0, or 0 for the plain softmax.  Key and value heads may differ in size.
@@ -73,7 +75,17 @@ __device__ __forceinline__ float block_max(float v, float* red) {
   return red[32];
 }
 
-// One warp per (token, head slot); the H query heads, then the G key heads, then the G value heads of the token.
+// What an attention mixer's inputs may have beyond the plain form: biases of the three projections, and query heads laid out in groups of
+// q_group >= H / G slots per key / value head (slots past the group's own heads are zeros).
+struct AppendExtras {
+  const float* bq;  // [H d] or null: added to the projection before everything else
+  const float* bk;  // [G d]
+  const float* bv;  // [G dv]
+  int q_group;
+  int has_kv;       // 0: there are no key / value projections (the layer reads another layer's cache)
+};
+
+// One warp per (token, head slot); the G q_group query slots, then the G key heads, then the G value heads of the token.
 template <typename T>
 __global__ void head_norm_rotary_append_kernel(const T* __restrict__ proj, long long ld, int q_col0, int k_col0, int v_col0,
                                                const float* __restrict__ wq, const float* __restrict__ wk, const double* __restrict__ freq,
@@ -81,47 +93,57 @@ __global__ void head_norm_rotary_append_kernel(const T* __restrict__ proj, long 
                                                const int* __restrict__ block_table, int bt_stride, int block_size, T* __restrict__ k_cache,
                                                long long k_block_stride, T* __restrict__ v_cache, long long v_block_stride, T* __restrict__ q_out,
                                                long long q_ld, int n_tokens, int H, int G, int d, int dv, int rot, float eps, int norm_v, int q_row,
-                                               int k_row, int v_row) {
+                                               int k_row, int v_row, AppendExtras ex) {
   const int gw = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-  const int per_tok = H + 2 * G;
+  const int n_q = G * ex.q_group, per_tok = n_q + (ex.has_kv ? 2 * G : 0);
   if (gw >= n_tokens * per_tok) return;
   const int t = gw / per_tok, slot = gw % per_tok;
   const int pos = tok_pos[t];
   const T* row = proj + static_cast<long long>(t) * ld;
   long long cache_row = 0;
-  if (slot >= H) cache_row = block_table[static_cast<size_t>(tok_seq[t]) * bt_stride + pos / block_size];
+  if (slot >= n_q) cache_row = block_table[static_cast<size_t>(tok_seq[t]) * bt_stride + pos / block_size];
   const int in_block = pos % block_size;
-  if (slot >= H + G) {  // a value head: its own root mean square, no weight
-    const int g = slot - H - G;
+  if (slot >= n_q + G) {  // a value head: its own root mean square, no weight
+    const int g = slot - n_q - G;
     const T* src = row + v_col0 + g * dv;
+    const float* bias = ex.bv ? ex.bv + g * dv : nullptr;
+    auto at = [&](int c) { return bias ? to_f(src[c]) + bias[c] : to_f(src[c]); };
     T* dst = v_cache + cache_row * v_block_stride + (static_cast<long long>(in_block) * G + g) * v_row;
     float inv = 1.f;
     if (norm_v) {
       float s = 0.f;
-      for (int c = lane; c < dv; c += 32) { const float v = to_f(src[c]); s += v * v; }
+      for (int c = lane; c < dv; c += 32) { const float v = at(c); s += v * v; }
       s = warp_sum(s);
       inv = 1.f / sqrtf(s / static_cast<float>(dv) + eps);
     }
-    for (int c = lane; c < dv; c += 32) dst[c] = from_f<T>(to_f(src[c]) * inv);
+    for (int c = lane; c < dv; c += 32) dst[c] = from_f<T>(at(c) * inv);
     for (int c = dv + lane; c < v_row; c += 32) dst[c] = from_f<T>(0.f);  // rows padded to a width the tensor-core kernels take
     return;
   }
-  const bool is_q = slot < H;
-  const int head = is_q ? slot : slot - H;
+  const bool is_q = slot < n_q;
+  const int per = H / G;
+  T* dst = is_q ? q_out + static_cast<long long>(t) * q_ld + slot * q_row
+                : k_cache + cache_row * k_block_stride + (static_cast<long long>(in_block) * G + (slot - n_q)) * k_row;
+  if (is_q && slot % ex.q_group >= per) {  // a slot without a head
+    for (int c = lane; c < q_row; c += 32) dst[c] = from_f<T>(0.f);
+    return;
+  }
+  const int head = is_q ? (slot / ex.q_group) * per + slot % ex.q_group : slot - n_q;
   const T* src = row + (is_q ? q_col0 : k_col0) + head * d;
   const float* w = is_q ? wq : wk;
-  T* dst = is_q ? q_out + static_cast<long long>(t) * q_ld + head * q_row
-                : k_cache + cache_row * k_block_stride + (static_cast<long long>(in_block) * G + head) * k_row;
+  const float* bias = is_q ? ex.bq : ex.bk;
+  if (bias) bias += head * d;
+  auto at = [&](int c) { return bias ? to_f(src[c]) + bias[c] : to_f(src[c]); };
   float inv = 1.f;
   if (w != nullptr) {
     float s = 0.f;
-    for (int c = lane; c < d; c += 32) { const float v = to_f(src[c]); s += v * v; }
+    for (int c = lane; c < d; c += 32) { const float v = at(c); s += v * v; }
     s = warp_sum(s);
     inv = 1.f / sqrtf(s / static_cast<float>(d) + eps);
   }
   const int half = rot >> 1;
   for (int i = lane; i < half; i += 32) {
-    const float u = to_f(src[i]) * inv * (w ? w[i] : 1.f), v = to_f(src[i + half]) * inv * (w ? w[i + half] : 1.f);
+    const float u = at(i) * inv * (w ? w[i] : 1.f), v = at(i + half) * inv * (w ? w[i + half] : 1.f);
     double a = static_cast<double>(pos) * freq[i];
     a -= 6.283185307179586476925 * rint(a * 0.15915494309189533576888);  // into [-pi, pi] before single precision takes over
     float sn, cs;
@@ -131,7 +153,7 @@ __global__ void head_norm_rotary_append_kernel(const T* __restrict__ proj, long 
     dst[i] = from_f<T>(u * cs - v * sn);
     dst[i + half] = from_f<T>(v * cs + u * sn);
   }
-  for (int c = rot + lane; c < d; c += 32) dst[c] = from_f<T>(to_f(src[c]) * inv * (w ? w[c] : 1.f));
+  for (int c = rot + lane; c < d; c += 32) dst[c] = from_f<T>(at(c) * inv * (w ? w[c] : 1.f));
   for (int c = d + lane; c < (is_q ? q_row : k_row); c += 32) dst[c] = from_f<T>(0.f);  // padding: adds nothing to a score
 }
 
@@ -142,6 +164,7 @@ struct SinkExtras {
   const float* r1;             // [H] or null: the score of key j loses r1[h] ln(1 + r2[h] (pos - j))
   const float* r2;
   int part;                    // > 0: a query at pos sees only the keys j <= pos with j / part == pos / part
+  int window;                  // > 0: a query at pos sees only the keys j <= pos with pos - j < window
   int k_row, v_row;            // elements between the heads of a cached key row / value row (>= d, dv)
   long long q_head_stride;     // elements between the heads of a query row
   long long out_head_stride;   // elements between the heads of an output row
@@ -166,7 +189,7 @@ sink_attention_kernel(const T* __restrict__ q, long long q_ld, const T* __restri
   for (int c = threadIdx.x; c < d; c += SA_THREADS) qs[c] = to_f(q[static_cast<long long>(t) * q_ld + h * ex.q_head_stride + c]) * scale;
   for (int c = threadIdx.x; c < dv; c += SA_THREADS) acc[c] = 0.f;
   const int n = pos + 1;
-  const int first = ex.part > 0 ? (pos / ex.part) * ex.part : 0;
+  const int first = max(ex.part > 0 ? (pos / ex.part) * ex.part : 0, ex.window > 0 ? pos + 1 - ex.window : 0);
   const int* bt = block_table + static_cast<size_t>(seq) * bt_stride;
   const float inv_cap = cap > 0.f ? 1.f / cap : 0.f;
   const float r1 = ex.r1 ? ex.r1[h] : 0.f, r2 = ex.r1 ? ex.r2[h] : 0.f;
@@ -463,29 +486,34 @@ using namespace dsb::sinkattn;
 // sine multiplied by `mag`.  Value heads: divided by their root mean square over dv when norm_v.  Queries -> q_out [T, q_ld]; keys ->
 // k_cache, values -> v_cache at the token's (block, slot) (see the file header for the plane addressing).  q_row / k_row / v_row: elements
 // between consecutive heads of a query row / a cached key row / a cached value row (>= d, d, dv); what lies past a head's own entries is
-// written as zeros, so that heads padded to a common width of 64 / 128 can be served by the tensor-core attention kernels.
+// written as zeros, so that heads padded to a common width of 64 / 128 can be served by the tensor-core attention kernels.  bq / bk / bv (fp32,
+// or null): biases added to the projections first.  q_group >= H / G: query head h goes to slot (h / (H / G)) q_group + h % (H / G) of its row,
+// slots without a head are zeros.  has_kv = 0: no key / value projections (the layer reads another layer's cache), only queries are prepared.
 DSB_EXPORT int dsb200_head_norm_rotary_append(const void* proj, long long ld, int q_col0, int k_col0, int v_col0, const float* wq, const float* wk,
                                               const double* freq, float mag, const int* tok_seq, const int* tok_pos, const int* block_table,
                                               int bt_stride, int block_size, void* k_cache, long long k_block_stride, void* v_cache,
                                               long long v_block_stride, void* q_out, long long q_ld, int n_tokens, int H, int G, int d, int dv,
-                                              int rot_dims, float eps, int norm_v, int q_row, int k_row, int v_row, int dtype, cudaStream_t stream) {
+                                              int rot_dims, float eps, int norm_v, int q_row, int k_row, int v_row, const float* bq, const float* bk,
+                                              const float* bv, int q_group, int has_kv, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
   DSB_REQUIRE(H >= 1 && G >= 1 && d >= 1 && dv >= 1 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= d && (rot_dims == 0 || freq != nullptr),
               "head_norm_rotary_append: heads %d / %d, head sizes %d / %d, rotated %d", H, G, d, dv, rot_dims);
   DSB_REQUIRE(q_row >= d && k_row >= d && v_row >= dv, "head_norm_rotary_append: row widths %d / %d / %d below the head sizes %d / %d", q_row, k_row, v_row, d, dv);
-  const long long warps = static_cast<long long>(n_tokens) * (H + 2 * G);
+  DSB_REQUIRE(H % G == 0 && q_group >= H / G, "head_norm_rotary_append: %d slots for the %d query heads of a key / value head", q_group, H / G);
+  const AppendExtras ex{bq, bk, bv, q_group, has_kv};
+  const long long warps = static_cast<long long>(n_tokens) * (G * q_group + (has_kv ? 2 * G : 0));
   const int wpb = 8;
   const int grid = static_cast<int>((warps + wpb - 1) / wpb);
   if (dtype == 0)
     head_norm_rotary_append_kernel<bf16><<<grid, wpb * 32, 0, stream>>>((const bf16*)proj, ld, q_col0, k_col0, v_col0, wq, wk, freq, mag, tok_seq, tok_pos,
                                                                        block_table, bt_stride, block_size, (bf16*)k_cache, k_block_stride,
                                                                        (bf16*)v_cache, v_block_stride, (bf16*)q_out, q_ld, n_tokens, H, G, d, dv,
-                                                                       rot_dims, eps, norm_v, q_row, k_row, v_row);
+                                                                       rot_dims, eps, norm_v, q_row, k_row, v_row, ex);
   else
     head_norm_rotary_append_kernel<float><<<grid, wpb * 32, 0, stream>>>((const float*)proj, ld, q_col0, k_col0, v_col0, wq, wk, freq, mag, tok_seq,
                                                                         tok_pos, block_table, bt_stride, block_size, (float*)k_cache, k_block_stride,
                                                                         (float*)v_cache, v_block_stride, (float*)q_out, q_ld, n_tokens, H, G, d, dv,
-                                                                        rot_dims, eps, norm_v, q_row, k_row, v_row);
+                                                                        rot_dims, eps, norm_v, q_row, k_row, v_row, ex);
   DSB_CHECK_CUDA(cudaGetLastError());
   return DSB_OK;
 }
@@ -518,26 +546,27 @@ DSB_EXPORT int dsb200_sink_attention(const void* q, long long q_ld, const void* 
   if (n_tokens == 0) return DSB_OK;
   DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && d >= 1 && dv >= 1 && d + dv <= 8192 && sink >= 0.f, "sink_attention: heads %d / %d, head sizes %d / %d", H, G,
               d, dv);
-  const SinkExtras ex{nullptr, nullptr, nullptr, 0, d, dv, d, dv};
+  const SinkExtras ex{nullptr, nullptr, nullptr, 0, 0, d, dv, d, dv};
   return launch_sink_attention(q, q_ld, k_cache, k_block_stride, v_cache, v_block_stride, tok_seq, tok_pos, block_table, bt_stride, block_size, out,
                                out_ld, n_tokens, H, G, d, dv, scale, cap, sink, ex, dtype, stream);
 }
 
 // `sink_attention` with learned sinks, a distance term, a mask by parts and free strides:
 //   sink_logit [H] (or null): exp(sink_logit[h]) joins head h's denominator;   r1, r2 [H] (or both null): s_j -= r1[h] ln(1 + r2[h] (pos - j));
-//   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible;
+//   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible; window > 0: only
+//   the keys with pos - j < window;
 //   q[t * q_ld + h * q_head_stride + c], out[t * out_ld + h * out_head_stride + c]; a cached key / value head starts every k_row / v_row
 //   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start).
 DSB_EXPORT int dsb200_sink_attention_ex(const void* q, long long q_ld, long long q_head_stride, const void* k_cache, long long k_block_stride, int k_row,
                                         const void* v_cache, long long v_block_stride, int v_row, const int* tok_seq, const int* tok_pos,
                                         const int* block_table, int bt_stride, int block_size, void* out, long long out_ld, long long out_head_stride,
                                         int n_tokens, int H, int G, int d, int dv, float scale, float cap, float sink, const float* sink_logit,
-                                        const float* r1, const float* r2, int part, int dtype, cudaStream_t stream) {
+                                        const float* r1, const float* r2, int part, int window, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
-  DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && d >= 1 && dv >= 1 && d + dv <= 8192 && sink >= 0.f && part >= 0 && k_row >= d && v_row >= dv &&
+  DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && d >= 1 && dv >= 1 && d + dv <= 8192 && sink >= 0.f && part >= 0 && window >= 0 && k_row >= d && v_row >= dv &&
                   (r1 == nullptr) == (r2 == nullptr),
               "sink_attention: heads %d / %d, head sizes %d / %d, rows %d / %d, part %d", H, G, d, dv, k_row, v_row, part);
-  const SinkExtras ex{sink_logit, r1, r2, part, k_row, v_row, q_head_stride, out_head_stride};
+  const SinkExtras ex{sink_logit, r1, r2, part, window, k_row, v_row, q_head_stride, out_head_stride};
   return launch_sink_attention(q, q_ld, k_cache, k_block_stride, v_cache, v_block_stride, tok_seq, tok_pos, block_table, bt_stride, block_size, out,
                                out_ld, n_tokens, H, G, d, dv, scale, cap, sink, ex, dtype, stream);
 }

@@ -7,6 +7,7 @@ import torch
 class NormTypeEnum(Enum):
     LayerNorm = "layer_norm"
     RMSNorm = "rms_norm"
+    DynamicTanh = "dynamic_tanh"  # tanh(alpha x) * w + b: no statistic of the row
 
 
 class DtypeEnum(Enum):

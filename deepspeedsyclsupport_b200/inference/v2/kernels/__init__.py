@@ -237,9 +237,10 @@ native.register_sigs({
     "dsb200_latent_attention": "p i ll p i p ll p ppp ii iii f i p",
     "dsb200_sigmoid_gate_mul": "p l p l l i i p",
     "dsb200_clamped_swish_gate": "pp l i fff i p",
-    "dsb200_clamped_swish_gate_cols": "p l ii p l l i fff i p",
+    "dsb200_clamped_swish_gate_cols": "p l iii p l l i fff i p",
+    "dsb200_stream_tanh_norm": "ppp i p ppp p i pp ii p",
     "dsb200_softcap": "p l l i f p",
-    "dsb200_grouped_topk_gating": "pppppp iiiiiii p",
+    "dsb200_grouped_topk_gating": "ppppppp iiiiiii p",
     "dsb200_moe_scatter_rows": "ppppppp iiii i p p",
     "dsb200_moe_gather_rows": "pppp iii i p i p p",
     "dsb200_moe_gemm_rows": "pppp iiii i p",
@@ -285,6 +286,25 @@ def stream_group_norm(x, branches=(), branch_fp32=None, w=None, groups=1, eps=1e
     native.check(native.lib().dsb200_stream_group_norm(native.ptr(x), native.ptr(ys[0]), native.ptr(ys[1]), _dt(ys[0]) if ys[0] is not None else 0,
                                                        native.ptr(branch_fp32), native.ptr(w), native.ptr(out), _DT[out_dtype], native.ptr(out32),
                                                        native.ptr(rows), n, x.shape[1], int(groups), float(eps), native.stream_ptr()))
+    if fp32_copy:
+        return out, (out32 if out32 is not None else out)
+    return out
+
+
+def stream_tanh_norm(x, branches=(), branch_fp32=None, alpha=None, w=None, b=None, out_dtype=torch.bfloat16, rows=None, fp32_copy=False):
+    """`stream_group_norm` with out = tanh(alpha x) * w + b in place of the RMS norm (alpha: one fp32 value on the device)."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.is_cuda and len(branches) <= 2
+    ys = [y if y.is_contiguous() else y.contiguous() for y in branches]
+    assert all(y.shape == x.shape and y.dtype == ys[0].dtype for y in ys)
+    assert branch_fp32 is None or (branch_fp32.shape == x.shape and branch_fp32.dtype == torch.float32 and branch_fp32.is_contiguous())
+    assert w is None or all(p.dtype == torch.float32 and p.is_cuda and p.numel() == n for p, n in ((w, x.shape[1]), (b, x.shape[1]), (alpha, 1)))
+    n = x.shape[0] if rows is None else rows.numel()
+    out = torch.empty(n, x.shape[1], dtype=out_dtype, device=x.device) if w is not None else None
+    out32 = torch.empty(n, x.shape[1], dtype=torch.float32, device=x.device) if (fp32_copy and w is not None and out_dtype != torch.float32) else None
+    ys += [None] * (2 - len(ys))
+    native.check(native.lib().dsb200_stream_tanh_norm(native.ptr(x), native.ptr(ys[0]), native.ptr(ys[1]), _dt(ys[0]) if ys[0] is not None else 0,
+                                                      native.ptr(branch_fp32), native.ptr(alpha), native.ptr(w), native.ptr(b), native.ptr(out),
+                                                      _DT[out_dtype], native.ptr(out32), native.ptr(rows), n, x.shape[1], native.stream_ptr()))
     if fp32_copy:
         return out, (out32 if out32 is not None else out)
     return out
@@ -415,11 +435,13 @@ def clamped_swish_gate(gu, alpha, limit, shift):
     return out
 
 
-def clamped_swish_gate_cols(gu, gate_col0, up_col0, F, out, alpha, limit, shift):
+def clamped_swish_gate_cols(gu, gate_col0, up_col0, F, out, alpha, limit, shift, row_gate_col=None):
     """`clamped_swish_gate` on column ranges: gate = gu[:, gate_col0 : gate_col0 + F], up = gu[:, up_col0 : up_col0 + F] of a fused projection,
-    result into `out` [rows, F] (a view with unit column stride, e.g. a column range of the next GEMM's input)."""
+    result into `out` [rows, F] (a view with unit column stride, e.g. a column range of the next GEMM's input).  `row_gate_col`: every row is also
+    multiplied by the sigmoid of the number gu holds in that column (one gate per token)."""
     assert gu.stride(1) == 1 and out.stride(1) == 1 and out.shape == (gu.shape[0], F) and gu.dtype == out.dtype
-    native.check(native.lib().dsb200_clamped_swish_gate_cols(native.ptr(gu), gu.stride(0), int(gate_col0), int(up_col0), native.ptr(out), out.stride(0),
+    native.check(native.lib().dsb200_clamped_swish_gate_cols(native.ptr(gu), gu.stride(0), int(gate_col0), int(up_col0),
+                                                             -1 if row_gate_col is None else int(row_gate_col), native.ptr(out), out.stride(0),
                                                              gu.shape[0], int(F), float(alpha), float(limit), float(shift), _dt(gu), native.stream_ptr()))
     return out
 
@@ -432,17 +454,18 @@ def softcap_(logits, cap):
     return logits
 
 
-def grouped_topk_gating(logits, k, correction=None, groups=1, keep=1, normalize=False, sigmoid_scores=False):
+def grouped_topk_gating(logits, k, correction=None, groups=1, keep=1, normalize=False, sigmoid_scores=False, bias=None):
     """Router with a selection bias and contiguous expert groups (see csrc/ragged/latent_ops.cu).  logits [T, E] fp32 ->
     (expert_counts [E] int32, scores [T, k] fp32, assignments [T, k] int32, offsets [T, k] int32), as `top_k_gating`.
-    `sigmoid_scores`: an expert's score is the sigmoid of its own logit instead of its softmax probability."""
+    `sigmoid_scores`: an expert's score is the sigmoid of its own logit instead of its softmax probability.  `bias` (fp32 [E]) joins the logits
+    first (it counts for the selection and for the weights)."""
     assert logits.dtype == torch.float32 and logits.is_cuda and logits.is_contiguous()
     T, E = logits.shape
     counts = torch.zeros(E, dtype=torch.int32, device=logits.device)
     scores = torch.empty(T, k, dtype=torch.float32, device=logits.device)
     asg = torch.empty(T, k, dtype=torch.int32, device=logits.device)
     off = torch.empty(T, k, dtype=torch.int32, device=logits.device)
-    native.check(native.lib().dsb200_grouped_topk_gating(native.ptr(logits), native.ptr(correction), native.ptr(counts), native.ptr(scores),
+    native.check(native.lib().dsb200_grouped_topk_gating(native.ptr(logits), native.ptr(bias), native.ptr(correction), native.ptr(counts), native.ptr(scores),
                                                          native.ptr(asg), native.ptr(off), T, E, k, groups, keep, int(normalize),
                                                          int(sigmoid_scores), native.stream_ptr()))
     return counts, scores, asg, off
@@ -501,10 +524,10 @@ native.register_sigs({
     "dsb200_delta_rule_scan": "ppppp p pp iiiii p",
     "dsb200_head_norm_gate": "pp i p l p l iii ff i p",
     "dsb200_tied_gate_scan": "p l iii pp p pp iiii i p",
-    "dsb200_head_norm_rotary_append": "p l iii pp p f ppp ii p l p l p l iiiii i f i iii i p",
+    "dsb200_head_norm_rotary_append": "p l iii pp p f ppp ii p l p l p l iiiii i f i iii ppp ii i p",
     "dsb200_sink_attention": "p l p l p l ppp ii p l iiiii fff i p",
     "dsb200_paged_flash_sink": "p l pp l ppp iiiiiii fff ii p i p",
-    "dsb200_paged_flash_sink_ex": "p l pp l ppp iiiiiii fff ppp i ii p i p",
+    "dsb200_paged_flash_sink_ex": "p l pp l ppp iiiiiii fff ppp ii ii p i p",
 }, restype_long=("dsb200_scan_state_floats", ))
 
 
@@ -664,19 +687,25 @@ def cache_planes(k_cache, v_cache=None):
 
 
 def head_norm_rotary_append(proj, q_col0, k_col0, v_col0, wq, wk, freq, mag, tok_seq, tok_pos, block_table, block_size, k_plane, v_plane, q_out,
-                            H, G, d, dv, rot_dims, eps, norm_v=True, row=None):
+                            H, G, d, dv, rot_dims, eps, norm_v=True, row=None, biases=None, q_group=None, kv=True):
     """Per-head RMS norm (weights wq / wk [d], shared by the heads) and rotation of the first rot_dims entries (entry i with entry
     i + rot_dims / 2, angle pos * freq[i], cosine and sine times `mag`) of the query / key heads in columns q_col0 / k_col0 of proj; value
     heads (columns v_col0) divided by their own root mean square when `norm_v`.  Queries -> q_out [T, >= H d]; keys / values -> their planes.
-    `row`: every query head, cached key head and cached value head occupies this many entries (>= d and dv), zeros behind its own."""
+    `row`: every query head, cached key head and cached value head occupies this many entries (>= d and dv), zeros behind its own.
+    `biases`: fp32 (q [H d], k [G d], v [G dv]) added to the projections first (None: none).  `q_group`: the query heads of a key / value head
+    occupy this many slots (>= H / G; zeros in the slots without a head).  `kv` False: only queries are prepared, the planes are left alone."""
     T = proj.shape[0]
+    bq, bk, bv = biases if biases is not None else (None, None, None)
+    for b, n in ((bq, H * d), (bk, G * d), (bv, G * dv)):
+        assert b is None or (b.dtype == torch.float32 and b.is_cuda and b.numel() == n)
     (kc, ks), (vc, vs) = k_plane, v_plane
     assert proj.stride(1) == 1 and q_out.stride(1) == 1 and q_out.dtype == proj.dtype == kc.dtype == vc.dtype
     native.check(native.lib().dsb200_head_norm_rotary_append(native.ptr(proj), proj.stride(0), q_col0, k_col0, v_col0, native.ptr(wq), native.ptr(wk),
                                                              native.ptr(freq), float(mag), native.ptr(tok_seq), native.ptr(tok_pos),
                                                              native.ptr(block_table), block_table.stride(0), int(block_size), native.ptr(kc), ks,
                                                              native.ptr(vc), vs, native.ptr(q_out), q_out.stride(0), T, H, G, d, dv, int(rot_dims),
-                                                             float(eps), int(norm_v), int(row or d), int(row or d), int(row or dv), _dt(proj),
+                                                             float(eps), int(norm_v), int(row or d), int(row or d), int(row or dv), native.ptr(bq),
+                                                             native.ptr(bk), native.ptr(bv), int(q_group or H // G), int(kv), _dt(proj),
                                                              native.stream_ptr()))
     return q_out
 
@@ -703,10 +732,11 @@ def paged_flash_sink_ok(q, cache, out, H, G, d, dv):
 
 
 def paged_flash_sink(q, cache, tok_seq, tok_pos, block_table, out, H, G, d, scale, softcap=0.0, sink=1.0, decode=False, max_context=None, n_splits=None,
-                     sink_logit=None, r1=None, r2=None, part=0):
+                     sink_logit=None, r1=None, r2=None, part=0, window=0):
     """`sink_attention` / `sink_attention_ex` on the tensor cores (csrc/attn/paged_flash.cu: TMA pages through the block table, S / P / O in
     TMEM) for a two-plane cache [blocks, 2, block_size, G, d].  `decode`: (almost) one token per sequence -- the small-atom kernel.
-    sink_logit / r1, r2 (fp32 [H]) / part: learned sinks, the logarithmic distance term and the mask by parts, as in `sink_attention_ex`."""
+    sink_logit / r1, r2 (fp32 [H]) / part: learned sinks, the logarithmic distance term and the mask by parts, as in `sink_attention_ex`;
+    `window` > 0: only the keys less than that far back (only their pages are visited)."""
     for p in (sink_logit, r1, r2):
         assert p is None or (p.dtype == torch.float32 and p.numel() == H and p.is_cuda)
     T = q.shape[0]
@@ -715,14 +745,15 @@ def paged_flash_sink(q, cache, tok_seq, tok_pos, block_table, out, H, G, d, scal
     nt = (16 if decode else 128) // group
     max_atoms = max(1, min(T, (T + nt - 1) // nt + block_table.shape[0]))
     if n_splits is None:
-        pages = -(-(max_context if max_context is not None else block_table.shape[1] * bs) // 128)
+        ctx = max_context if max_context is not None else block_table.shape[1] * bs
+        pages = -(-(min(ctx, window + 256) if window > 0 else ctx) // 128)
         n_splits = _pick_splits(T, H, d, max_atoms * G, pages, page_us=0.45 if decode else 0.7)
     nbytes = native.lib().dsb200_paged_flash_scratch_bytes(T, H, d, max_atoms, n_splits)
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
     native.check(native.lib().dsb200_paged_flash_sink_ex(native.ptr(q), q.stride(0), native.ptr(cache), native.ptr(out), out.stride(0), native.ptr(tok_seq),
                                                          native.ptr(tok_pos), native.ptr(block_table), T, H, G, d, bs, block_table.shape[1],
                                                          cache.shape[0], float(scale), float(softcap), float(sink), native.ptr(sink_logit),
-                                                         native.ptr(r1), native.ptr(r2), int(part), max_atoms, n_splits, native.ptr(scratch),
+                                                         native.ptr(r1), native.ptr(r2), int(part), int(window), max_atoms, n_splits, native.ptr(scratch),
                                                          int(decode), native.stream_ptr()), 2 + (n_splits > 1))
     return out
 
@@ -736,7 +767,7 @@ native.register_sigs({
     "dsb200_gate_heads_scalar": "pp l p l iii i p",
     "dsb200_mingru_scratch_floats": "iii",
     "dsb200_mingru_scan": "p l iii pp pp p p l iii i p i p",
-    "dsb200_sink_attention_ex": "p l l p l i p l i ppp ii p l l iiiii fff ppp i i p",
+    "dsb200_sink_attention_ex": "p l l p l i p l i ppp ii p l l iiiii fff ppp ii i p",
     "dsb200_latent_rotary_append": "p l ii pp ppp ii p i iiiii i f i p",
     "dsb200_conv_head_norm_append": "p l i pppp p pppp ii p l p l p l p p p iiiiii f iii i p",
 }, restype_long=("dsb200_mingru_scratch_floats", ))
@@ -805,10 +836,10 @@ def mingru_scan(proj, z_col0, x_col0, g_col0, z_bias, x_bias, tok_seq, seq_desc,
 
 
 def sink_attention_ex(q, q_head_stride, k_plane, k_row, v_plane, v_row, tok_seq, tok_pos, block_table, block_size, out, out_head_stride, H, G, d, dv,
-                      scale, softcap=0.0, sink=0.0, sink_logit=None, r1=None, r2=None, part=0):
+                      scale, softcap=0.0, sink=0.0, sink_logit=None, r1=None, r2=None, part=0, window=0):
     """`sink_attention` with learned sinks (sink_logit fp32 [H]: exp of it joins the head's denominator), a distance term (r1, r2 fp32 [H]: the
     score of key j loses r1 ln(1 + r2 (pos - j))), a mask by parts (`part` > 0: a query sees only the keys of its own part of that many
-    positions, counted from the sequence's start) and free strides: q / out are addressed [t * stride(0) + h * head_stride + c], a cached
+    positions, counted from the sequence's start), a sliding window (`window` > 0: only keys less than that far back) and free strides: q / out are addressed [t * stride(0) + h * head_stride + c], a cached
     key / value head starts every k_row / v_row elements of its token's row."""
     T = q.shape[0]
     (kc, ks), (vc, vs) = k_plane, v_plane
@@ -819,7 +850,7 @@ def sink_attention_ex(q, q_head_stride, k_plane, k_row, v_plane, v_row, tok_seq,
                                                        int(v_row), native.ptr(tok_seq), native.ptr(tok_pos), native.ptr(block_table),
                                                        block_table.stride(0), int(block_size), native.ptr(out), out.stride(0), int(out_head_stride), T,
                                                        H, G, d, dv, float(scale), float(softcap), float(sink), native.ptr(sink_logit), native.ptr(r1),
-                                                       native.ptr(r2), int(part), _dt(q), native.stream_ptr()))
+                                                       native.ptr(r2), int(part), int(window), _dt(q), native.stream_ptr()))
     return out
 
 
@@ -855,3 +886,53 @@ def conv_head_norm_append(proj, col0, bias, conv_w, wq, wk, state, seq_desc, tok
                                                            native.ptr(v_other), native.ptr(mix), native.ptr(v_own), proj.shape[0], H, G, d, dv, int(taps),
                                                            float(eps), int(row or d), int(row or d), int(row or dv), _dt(proj), native.stream_ptr()))
     return q_out
+
+
+# ---- kernels of csrc/ragged/ssd_ops.cu: state-space mixers with one decay per head
+native.register_sigs({
+    "dsb200_ssd_prepare": "p l ii ppp pp pp ppp iiii i p",
+    "dsb200_ssd_scan": "ppppp pp iiiii ii i p",
+    "dsb200_gated_group_norm": "pp l pp l iii f i p",
+})
+
+
+def ssd_prepare(proj, col0, dt_col0, conv_w, conv_b, state, seq_desc, tok_seq, dt_bias, rate, C, H, taps):
+    """Columns col0 .. + C of proj -> xbc [T, C] = silu(conv_b + causal convolution over time) (conv_w fp32 [taps, C]; rows before this step's
+    come from state [slots, taps - 1, C], rows before the sequence are zeros); columns dt_col0 .. + H -> fp32 (dt [T, H] = softplus(pre + dt_bias),
+    la [T, H] = -rate dt).  Follow with `conv_state_update`."""
+    T = proj.shape[0]
+    assert proj.stride(1) == 1 and conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape == (taps, C) and conv_b.numel() == C
+    assert state is None or (state.dtype == proj.dtype and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, C))
+    for p, n in ((conv_b, C), (dt_bias, H), (rate, H)):
+        assert p.dtype == torch.float32 and p.numel() == n and p.is_cuda
+    xbc = torch.empty(T, C, dtype=proj.dtype, device=proj.device)
+    dt = torch.empty(T, H, dtype=torch.float32, device=proj.device)
+    la = torch.empty(T, H, dtype=torch.float32, device=proj.device)
+    native.check(native.lib().dsb200_ssd_prepare(native.ptr(proj), proj.stride(0), int(col0), int(dt_col0), native.ptr(conv_w), native.ptr(conv_b),
+                                                 native.ptr(state), native.ptr(seq_desc), native.ptr(tok_seq), native.ptr(dt_bias), native.ptr(rate),
+                                                 native.ptr(xbc), native.ptr(dt), native.ptr(la), T, C, H, int(taps), _dt(proj), native.stream_ptr()))
+    return xbc, dt, la
+
+
+def ssd_scan(xbc, dt, la, D, seq_desc, n_seqs, state, H, G, N, P, out=None, min_new=1, max_new=2**31 - 1):
+    """S <- exp(la) S + dt B x^T, y = S^T C + D x per head over every sequence's new tokens in order (sequences with min_new .. max_new of them)
+    -> fp32 [T, H P].  xbc [T, H P + 2 G N] = (x | B | C); state fp32 [slots, H, N, P], updated in place."""
+    T = xbc.shape[0]
+    assert xbc.is_contiguous() and xbc.shape[1] == H * P + 2 * G * N and D.dtype == torch.float32 and D.numel() == H
+    assert all(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, H) for t in (dt, la))
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, P)
+    if out is None:
+        out = torch.empty(T, H * P, dtype=torch.float32, device=xbc.device)
+    native.check(native.lib().dsb200_ssd_scan(native.ptr(xbc), native.ptr(dt), native.ptr(la), native.ptr(D), native.ptr(seq_desc), native.ptr(state),
+                                              native.ptr(out), n_seqs, H, G, N, P, int(min_new), int(max_new), _dt(xbc), native.stream_ptr()))
+    return out
+
+
+def gated_group_norm(y, z, w, out, groups, eps):
+    """out = rms_norm_in_groups(y * silu(z)) * w: y fp32 [T, inner], z a view [T, inner] of the activation dtype, w fp32 [inner], out a view."""
+    T, inner = y.shape
+    assert y.dtype == torch.float32 and y.is_contiguous() and z.shape == y.shape == out.shape and z.stride(1) == 1 and out.stride(1) == 1
+    assert z.dtype == out.dtype and w.dtype == torch.float32 and w.numel() == inner
+    native.check(native.lib().dsb200_gated_group_norm(native.ptr(y), native.ptr(z), z.stride(0), native.ptr(w), native.ptr(out), out.stride(0), T, inner,
+                                                      int(groups), float(eps), _dt(z), native.stream_ptr()))
+    return out

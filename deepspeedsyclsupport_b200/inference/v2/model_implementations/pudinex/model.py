@@ -274,10 +274,8 @@ class PudinexInferenceModel(RaggedTransformer, DSInferenceModelBase):
             elif f is not None and f.shared_ff:
                 side_in, side_out = c["shared_in_w"], c["shared_down_w"]
             o_w = c["o_w"]
-            if L.kind == "attention" and self.attn_mods[i].out_head_width != L.attn.vdim:
-                # the attention kernels work on heads padded to a common width: zero weights meet the (zero) padding columns of their output
-                P = self.attn_mods[i].out_head_width
-                o_w = torch.nn.functional.pad(o_w.view(o_w.shape[0], L.attn.heads, L.attn.vdim), (0, P - L.attn.vdim)).reshape(o_w.shape[0], L.attn.heads * P)
+            if L.kind == "attention":  # zero weights meet the padding the attention kernels leave between heads
+                o_w = self.attn_mods[i].layout_output_weight(o_w)
             if side_in is None:
                 self._fused[i] = (c["mix_in_w"], o_w.contiguous())
             else:

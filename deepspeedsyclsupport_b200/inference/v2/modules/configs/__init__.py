@@ -4,5 +4,5 @@ from .embedding_config import DSEmbeddingsConfig
 from .linear_config import DSLinearConfig
 from .moe_config import DSMoEConfig
 from .norm_config import DSNormConfig
-from .recurrent_configs import DSDeltaRuleConfig, DSMatrixMemoryConfig, DSMinGRUConfig, DSTiedGateConfig
+from .recurrent_configs import DSDeltaRuleConfig, DSMatrixMemoryConfig, DSMinGRUConfig, DSStateSpaceConfig, DSTiedGateConfig
 from .unembed_config import DSUnembedConfig

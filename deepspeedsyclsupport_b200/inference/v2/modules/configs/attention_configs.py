@@ -145,7 +145,8 @@ class DSSinkAttentionConfig(DSModuleConfig):
     """Causal attention with per-head query / key RMS norms (one weight of head size shared by the heads, applied before the rotation), a
     rotate-half rotation of the first `rotate_dim` entries of a head, values divided by their own root mean square (no weight; cached so),
     scores scale * q . k soft-capped as softcap tanh(. / softcap), and a softmax whose denominator has `sink` added (1: one more entry of
-    score 0 without a value).  Query / key heads have `head_size` entries, value heads `value_size`."""
+    score 0 without a value; 0: the plain softmax).  Query / key heads have `head_size` entries, value heads `value_size`.  The norms and the cap
+    are optional; the projections may have biases (handed to the module's forward); the causal mask may be a sliding window."""
     n_heads_q: int
     n_heads_kv: int
     head_size: int
@@ -158,6 +159,8 @@ class DSSinkAttentionConfig(DSModuleConfig):
     rotate_dim: int = 0
     theta_base: float = 10_000.0
     rotary_scaling: Optional[RampRotaryScalingConfig] = None
+    window: int = 0  # > 0: a query sees only the keys less than this far back (itself and the window - 1 tokens before it)
+    reads_cache: bool = False  # the layer has no keys and values: it reads what another layer of equal head sizes wrote to ITS cache
     eps: float = 1e-6
     max_sequences: int
     input_dtype: DtypeEnum = DtypeEnum.bf16
@@ -173,6 +176,8 @@ class DSSinkAttentionConfig(DSModuleConfig):
             raise ValueError(f"rotate_dim must be even and at most head_size ({self.head_size}), got {self.rotate_dim}")
         if self.softcap < 0 or self.sink < 0:
             raise ValueError("softcap and sink cannot be negative")
+        if self.window < 0:
+            raise ValueError(f"window cannot be negative, got {self.window}")
         return self
 
     @property

@@ -18,6 +18,8 @@ class DSMoEConfig(DSModuleConfig):
     n_groups: int = 1
     keep_groups: int = 1
     use_correction: bool = False
+    # the router logits get a bias per expert (it counts for the selection AND for the weights)
+    router_bias: bool = False
     # how a router logit becomes a score: "softmax" over the experts, or "sigmoid" of every logit on its own
     score_function: str = "softmax"
     # True: the chosen expert's score multiplies the expert's INPUT (out = sum_k expert_k(s_k h)) instead of its output

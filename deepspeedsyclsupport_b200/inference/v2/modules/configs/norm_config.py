@@ -8,7 +8,7 @@ from ..ds_module import DSModuleConfig
 class DSNormConfig(DSModuleConfig):
     """One config serves DSPreNormBase and DSPostNormBase.  `residual_dtype` is the dtype of the residual stream the norm adds into,
     `input_dtype` that of the incoming hidden states, `output_dtype` that of the normalised result."""
-    type: NormTypeEnum  # layer_norm | rms_norm
+    type: NormTypeEnum  # layer_norm | rms_norm | dynamic_tanh (its eps is not used)
     channels: int  # width of the normalised (last) dimension
     eps: float = 1e-5
     residual_dtype: DtypeEnum = DtypeEnum.fp16

@@ -1,4 +1,6 @@
 """Configuration of the recurrent token mixers: layers that carry a fixed-size state per sequence instead of a growing cache."""
+from pydantic import model_validator
+
 from ...inference_utils import DtypeEnum
 from ..ds_module import DSModuleConfig
 
@@ -46,6 +48,33 @@ class DSTiedGateConfig(DSModuleConfig):
     max_sequences: int
     input_dtype: DtypeEnum = DtypeEnum.bf16
     output_dtype: DtypeEnum = DtypeEnum.bf16
+
+
+class DSStateSpaceConfig(DSModuleConfig):
+    """State-space mixer with one decay per head: the inputs x, B and C pass a short causal convolution (with bias) and silu;
+    dt = softplus(pre + dt_bias), S <- exp(-rate dt) S + dt B x^T (state_size x value_size per head, B and C shared by the heads of a group),
+    y = S^T C + D x; then y silu(z), an RMS norm in `norm_groups` equal parts of the whole row and a weight."""
+    n_heads: int
+    value_size: int
+    state_size: int
+    n_groups: int = 1
+    conv_taps: int = 4  # the last taps - 1 rows in front of the convolution are state
+    norm_groups: int = 1
+    eps: float = 1e-6
+    max_sequences: int
+    input_dtype: DtypeEnum = DtypeEnum.bf16
+    output_dtype: DtypeEnum = DtypeEnum.bf16
+
+    @model_validator(mode="after")
+    def _consistent(self):
+        for k in ("n_heads", "value_size", "state_size", "n_groups", "conv_taps", "norm_groups"):
+            if getattr(self, k) < 1:
+                raise ValueError(f"{k} must be positive")
+        if self.n_heads % self.n_groups != 0:
+            raise ValueError(f"{self.n_heads} heads do not split into {self.n_groups} groups")
+        if (self.n_heads * self.value_size) % self.norm_groups != 0:
+            raise ValueError(f"{self.n_heads * self.value_size} values do not split into {self.norm_groups} parts")
+        return self
 
 
 class DSMinGRUConfig(DSModuleConfig):

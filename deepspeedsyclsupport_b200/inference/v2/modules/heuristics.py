@@ -6,7 +6,7 @@ from ..inference_utils import ActivationType, NormTypeEnum
 from . import implementations  # noqa: F401  (registers the implementations)
 from .configs import (DSConvSinkAttentionConfig, DSDeltaRuleConfig, DSEmbeddingsConfig, DSLatentAttentionConfig, DSLinearConfig, DSMatrixMemoryConfig,
                       DSMinGRUConfig, DSMoEConfig, DSNormConfig, DSRotaryLatentAttentionConfig, DSSelfAttentionConfig, DSSinkAttentionConfig,
-                      DSTiedGateConfig, DSUnembedConfig, DSWindowedAttentionConfig)
+                      DSStateSpaceConfig, DSTiedGateConfig, DSUnembedConfig, DSWindowedAttentionConfig)
 from .interfaces import (DSEmbeddingBase, DSEmbeddingRegistry, DSLinearBase, DSLinearRegistry, DSMoEBase, DSMoERegistry, DSPostNormBase,
                          DSPostNormRegistry, DSPreNormBase, DSPreNormRegistry, DSRecurrentMixerBase, DSRecurrentRegistry, DSSelfAttentionBase,
                          DSSelfAttentionRegistry, DSUnembedBase, DSUnembedRegistry)
@@ -35,7 +35,7 @@ def instantiate_attention(attention_config, engine_config: RaggedInferenceEngine
 def instantiate_recurrent(mixer_config, engine_config: RaggedInferenceEngineConfig = None) -> DSRecurrentMixerBase:
     """Token mixers with a fixed-size state per sequence; the config class names the recurrence."""
     name = {DSMatrixMemoryConfig: "matrix_memory", DSDeltaRuleConfig: "channel_delta_rule", DSTiedGateConfig: "tied_gate_linear",
-            DSMinGRUConfig: "min_gru"}[type(mixer_config)]
+            DSMinGRUConfig: "min_gru", DSStateSpaceConfig: "state_space"}[type(mixer_config)]
     return DSRecurrentRegistry.instantiate_config(ConfigBundle(name=name, config=mixer_config))
 
 
@@ -58,7 +58,8 @@ def instantiate_linear(linear_config: DSLinearConfig, engine_config: RaggedInfer
 
 def instantiate_moe(moe_config: DSMoEConfig, engine_config: RaggedInferenceEngineConfig = None) -> DSMoEBase:
     if (moe_config.n_groups > 1 or moe_config.use_correction or ActivationType(moe_config.activation) == ActivationType.ClampedSwiGLU or
-            moe_config.score_function != "softmax" or moe_config.scale_input or moe_config.n_identity_experts > 0 or moe_config.fp32_combine):
+            moe_config.score_function != "softmax" or moe_config.scale_input or moe_config.n_identity_experts > 0 or moe_config.fp32_combine or
+            moe_config.router_bias):
         return DSMoERegistry.instantiate_config(ConfigBundle(name="grouped_topk_moe", config=moe_config))
     bundle = ConfigBundle(name="cutlass_multi_gemm_moe", config=moe_config, implementation_config={"weight_dtype": moe_config.input_dtype})
     return DSMoERegistry.instantiate_config(bundle)
@@ -74,6 +75,8 @@ def instantiate_pre_norm(norm_config: DSNormConfig, engine_config: RaggedInferen
     name = "cuda_pre_ln" if kind == NormTypeEnum.LayerNorm else ("cuda_sandwich_rms" if norm_config.sandwich else "cuda_pre_rms")
     if kind == NormTypeEnum.RMSNorm and norm_config.shared_input:
         name = "cuda_group_rms"
+    elif kind == NormTypeEnum.DynamicTanh:
+        name = "cuda_dynamic_tanh"
     return DSPreNormRegistry.instantiate_config(ConfigBundle(name=name, config=norm_config))
 
 

@@ -1,6 +1,6 @@
 """Mixture-of-experts MLP with a configurable fp32 router and a gated activation.
 
-Router (fp32): scores = softmax(W_r h) over all experts, or (`score_function` "sigmoid") the sigmoid of every logit on its own; the
+Router (fp32): scores = softmax(W_r h), or softmax(W_r h + b) with `router_bias`, over all experts, or (`score_function` "sigmoid") the sigmoid of every logit on its own; the
 SELECTION uses scores + correction (when the config has one), restricted to the `keep_groups` contiguous expert groups whose best
 selection score is largest; the WEIGHTS are the plain scores of the chosen experts (optionally renormalised).  They multiply the
 experts' outputs in the combine or, with `scale_input`, the experts' inputs in the scatter (out = sum_k expert_k(s_k h)).  `n_identity_experts`: the router has that many outputs more than there are
@@ -66,15 +66,15 @@ class DSGroupedTopKMoE(DSMoEBase):
 
     def forward(self, hidden_states: torch.Tensor, gate_w: torch.Tensor, mlp_1_w: torch.Tensor, mlp_2_w: torch.Tensor,
                 mlp_1_b: Optional[torch.Tensor] = None, mlp_2_b: Optional[torch.Tensor] = None,
-                correction: Optional[torch.Tensor] = None, router_input: Optional[torch.Tensor] = None) -> torch.Tensor:
+                correction: Optional[torch.Tensor] = None, router_bias: Optional[torch.Tensor] = None, router_input: Optional[torch.Tensor] = None) -> torch.Tensor:
         """`router_input`: fp32 [tokens, model_dim], the hidden states before their rounding to the activation dtype (the norm in front
         can emit them in the same pass); without it the router reads the rounded hidden states."""
         c = self._config
         assert mlp_1_b is None and mlp_2_b is None, "these experts have no biases"
-        assert (correction is not None) == c.use_correction
+        assert (correction is not None) == c.use_correction and (router_bias is not None) == c.router_bias
         logits = dense_matmul(router_input if router_input is not None else hidden_states.float(), gate_w)  # fp32 router logits
         counts, scores, assignments, offsets = K.grouped_topk_gating(logits, c.top_k, correction, c.n_groups, c.keep_groups, c.normalize_scores,
-                                                                     sigmoid_scores=c.score_function == "sigmoid")
+                                                                     sigmoid_scores=c.score_function == "sigmoid", bias=router_bias)
         moe_in, cumsum, slots = K.moe_scatter_rows(hidden_states, counts, assignments, offsets, row_scale=scores if c.scale_input else None)
         identity = None
         if c.n_identity_experts:  # their rows sit behind the last real expert's in the sorted order: the GEMMs never touch them, the combine

@@ -1,3 +1,4 @@
+from .cuda_dynamic_tanh import DSDynamicTanhNorm
 from .cuda_group_rms import DSGroupRMSNorm
 from .cuda_pre_ln import DSPreLNCUDAModule
 from .cuda_pre_rms import DSPreRMSCUDAModule

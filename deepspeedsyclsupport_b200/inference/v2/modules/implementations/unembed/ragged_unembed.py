@@ -37,7 +37,7 @@ class DSRaggedUnembed(DSUnembedBase):
 
     def forward(self, hidden_states: torch.Tensor, vocab_embedding: torch.Tensor, ragged_metadata, bias: Optional[torch.Tensor] = None,
                 gamma: Optional[torch.Tensor] = None, beta: Optional[torch.Tensor] = None,
-                residual: Optional[torch.Tensor] = None, pending=None) -> torch.Tensor:
+                residual: Optional[torch.Tensor] = None, pending=None, alpha: Optional[torch.Tensor] = None) -> torch.Tensor:
         """`residual` (optional): the residual stream the last hidden state still has to be added to -- only the gathered rows
         (one per sequence) are added and normalised, not the whole batch.  `pending` (fp32 stream only): ((outputs in the activation
         dtype, ...), fp32 output or None) of the last layer's sublayers that have not joined the stream yet; they are added to the
@@ -45,7 +45,7 @@ class DSRaggedUnembed(DSUnembedBase):
         last_tok = ragged_metadata.logit_rows()
         c = self._config
         if c.residual_fp32:
-            return self._forward_fp32_residual(hidden_states, vocab_embedding, last_tok, gamma, pending)
+            return self._forward_fp32_residual(hidden_states, vocab_embedding, last_tok, gamma, pending, beta, alpha)
         h = K.logits_gather(hidden_states, last_tok)
         r = K.logits_gather(residual, last_tok) if residual is not None else None
         if self._norm == NormTypeEnum.RMSNorm:
@@ -67,15 +67,18 @@ class DSRaggedUnembed(DSUnembedBase):
         self._output = logits
         return logits
 
-    def _forward_fp32_residual(self, residual, vocab_embedding, rows, gamma, pending=None):
-        """Gather + RMS norm of the wanted rows in one kernel (fp32 in, activation dtype out), projection with fp32 logits,
+    def _forward_fp32_residual(self, residual, vocab_embedding, rows, gamma, pending=None, beta=None, alpha=None):
+        """Gather + RMS norm (or tanh(alpha x) * gamma + beta) of the wanted rows in one kernel (fp32 in, activation dtype out), projection with fp32 logits,
         soft cap in place."""
         c = self._config
-        assert self._norm == NormTypeEnum.RMSNorm and residual.dtype == torch.float32
+        assert self._norm in (NormTypeEnum.RMSNorm, NormTypeEnum.DynamicTanh) and residual.dtype == torch.float32
         act = DtypeEnum(c.dtype).value
         if rows.numel() == 0:
             return torch.empty(0, vocab_embedding.shape[0], dtype=torch.float32, device=residual.device)
-        if c.norm_groups > 1 or pending is not None:  # the stream still lacks the last layer's outputs and / or is normed in parts
+        if self._norm == NormTypeEnum.DynamicTanh:
+            branches, fp32_branch = pending if pending is not None else ((), None)
+            h = K.stream_tanh_norm(residual, branches, fp32_branch, alpha, gamma, beta, out_dtype=act, rows=rows)
+        elif c.norm_groups > 1 or pending is not None:  # the stream still lacks the last layer's outputs and / or is normed in parts
             assert c.norm_weight_offset == 0.0
             branches, fp32_branch = pending if pending is not None else ((), None)
             h = K.stream_group_norm(residual, branches, fp32_branch, gamma, c.norm_groups, c.eps, out_dtype=act, rows=rows)

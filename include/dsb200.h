@@ -176,13 +176,14 @@ int dsb200_paged_flash_window(const void* q, long long q_tok_stride, const void*
  * bf16 at q_tok_stride elements per token (a multiple of 8), kv_cache [num_blocks][2][block_size][hkv][head_dim] bf16; out rows at out_ld
  * elements per token (a multiple of 8).  decode != 0 selects the small-atom kernel (head_dim 128, q:kv head ratios dividing 16).
  * sink_logit (hq floats): learned sinks, exp(sink_logit[h]) joins head h's denominator; r1, r2 (hq floats each): the score of key j for the
- * query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions.  Each may
- * be absent (null / 0). */
+ * query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions;
+ * window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0). */
 int dsb200_paged_flash_sink_ex(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld,
                                const int* tok_seq, const int* tok_pos, const int* block_table, int n_tokens, int hq,
                                int hkv, int head_dim, int block_size, int max_blocks_per_seq, int num_blocks, float scale,
                                float softcap, float sink, const float* sink_logit, const float* r1, const float* r2,
-                               int part, int max_atoms, int n_splits, void* scratch, int decode, dsb200_stream_t stream);
+                               int part, int window, int max_atoms, int n_splits, void* scratch, int decode,
+                               dsb200_stream_t stream);
 int dsb200_paged_flash_sink(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld,
                             const int* tok_seq, const int* tok_pos, const int* block_table, int n_tokens, int hq, int hkv,
                             int head_dim, int block_size, int max_blocks_per_seq, int num_blocks, float scale,
@@ -419,6 +420,10 @@ int dsb200_sandwich_norm(float* x, const void* y, int y_dtype, const float* wb, 
 int dsb200_stream_group_norm(float* x, const void* y0, const void* y1, int y_dtype, const float* y2, const float* w,
                              void* out, int out_dtype, float* out32, const int* rows, int n_rows, int dim, int groups,
                              float eps, dsb200_stream_t stream);
+/* `dsb200_stream_group_norm` with out[r] = tanh(alpha * row) * w + b in place of the RMS norm: alpha one float on the device, w and b [dim]. */
+int dsb200_stream_tanh_norm(float* x, const void* y0, const void* y1, int y_dtype, const float* y2, const float* alpha,
+                            const float* w, const float* b, void* out, int out_dtype, float* out32, const int* rows,
+                            int n_rows, int dim, dsb200_stream_t stream);
 /* lat [n_tokens, ld] holds (query latent [nq] | key/value latent [nkv]) of every token.  cq [n_tokens, nq] = plain-weight RMS norm
  * of the first part; the RMS-normed second part is written to the token's row of cache [blocks, block_size, cache_ld] (cache_ld >= nkv:
  * rows may be padded to a width the tensor-core attention takes; the padding is never written). */
@@ -446,20 +451,22 @@ int dsb200_gate_heads(const void* a, const void* g, long long g_ld, void* out, i
 int dsb200_clamped_swish_gate(const void* gu, void* out, long long rows, int F, float alpha, float limit, float shift,
                               int dtype, dsb200_stream_t stream);
 /* out[r, c] = g' * sigmoid(alpha g') * (clamp(u, -limit, limit) + shift) with g' = min(gu[r, gate_col0 + c], limit), u = gu[r, up_col0 + c], c < F:
- * gate and up are column ranges of one fused projection gu [rows, ld]; out [rows, out_ld] may be a column range of a wider buffer. */
-int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, void* out, long long out_ld,
-                                   long long rows, int F, float alpha, float limit, float shift, int dtype,
-                                   dsb200_stream_t stream);
+ * gate and up are column ranges of one fused projection gu [rows, ld]; out [rows, out_ld] may be a column range of a wider buffer.
+ * row_col >= 0: row r is also multiplied by sigmoid(gu[r, row_col]). */
+int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, int row_col, void* out,
+                                   long long out_ld, long long rows, int F, float alpha, float limit, float shift,
+                                   int dtype, dsb200_stream_t stream);
 /* x[r, c] = cap * tanh(x[r, c] / cap) over fp32 [rows, cols] with row stride ld */
 int dsb200_softcap(float* x, long long ld, long long rows, int cols, float cap, dsb200_stream_t stream);
-/* Router: scores = softmax over the E logits of a token, or (sigmoid_scores) the sigmoid of every logit on its own; selection score =
+/* Router: scores = softmax over the E logits of a token (bias[e], when given, joins the logits first), or (sigmoid_scores) the sigmoid of every
+ * logit on its own; selection score =
  * score + correction[e] (correction may be null); experts are split
  * into `groups` contiguous groups of equal size, of which the `keep` with the largest maximal selection score stay selectable; the top_k
  * selectable experts by selection score are assigned; their weights are the uncorrected scores (divided by their sum when
  * `normalize`).  Outputs as dsb200_top_k_gating; expert_counts must be zeroed by the caller. */
-int dsb200_grouped_topk_gating(const float* logits, const float* correction, int* expert_counts, float* scores,
-                               int* assignments, int* offsets, int n_tokens, int n_experts, int top_k, int groups,
-                               int keep, int normalize, int sigmoid_scores, dsb200_stream_t stream);
+int dsb200_grouped_topk_gating(const float* logits, const float* bias, const float* correction, int* expert_counts,
+                               float* scores, int* assignments, int* offsets, int n_tokens, int n_experts, int top_k,
+                               int groups, int keep, int normalize, int sigmoid_scores, dsb200_stream_t stream);
 /* Rows of x [n_tokens, dim] copied into expert-sorted order (any dim; dtype 0 = bf16, 1 = fp32); also writes the inclusive
  * per-expert row cumsum and every (token, k)'s row.  row_scale (optional, fp32 [n_tokens, top_k]): copy k of token t is multiplied by
  * row_scale[t, k] (routers whose weight applies to the expert's input). */
@@ -590,13 +597,16 @@ int dsb200_mingru_scan(const void* proj, long long ld, int z_col0, int x_col0, i
  * sine multiplied by `mag`.  Value heads: divided by their root mean square over dv when norm_v.  Queries -> q_out [T, q_ld]; keys ->
  * k_cache, values -> v_cache at the token's (block, slot) (see the file header for the plane addressing).  q_row / k_row / v_row: elements
  * between consecutive heads of a query row / a cached key row / a cached value row (>= d, d, dv); what lies past a head's own entries is
- * written as zeros, so that heads padded to a common width of 64 / 128 can be served by the tensor-core attention kernels. */
+ * written as zeros, so that heads padded to a common width of 64 / 128 can be served by the tensor-core attention kernels.  bq / bk / bv (fp32,
+ * or null): biases added to the projections first.  q_group >= H / G: query head h goes to slot (h / (H / G)) q_group + h % (H / G) of its row,
+ * slots without a head are zeros.  has_kv = 0: no key / value projections (the layer reads another layer's cache), only queries are prepared. */
 int dsb200_head_norm_rotary_append(const void* proj, long long ld, int q_col0, int k_col0, int v_col0, const float* wq,
                                    const float* wk, const double* freq, float mag, const int* tok_seq, const int* tok_pos,
                                    const int* block_table, int bt_stride, int block_size, void* k_cache,
                                    long long k_block_stride, void* v_cache, long long v_block_stride, void* q_out,
                                    long long q_ld, int n_tokens, int H, int G, int d, int dv, int rot_dims, float eps,
-                                   int norm_v, int q_row, int k_row, int v_row, int dtype, dsb200_stream_t stream);
+                                   int norm_v, int q_row, int k_row, int v_row, const float* bq, const float* bk,
+                                   const float* bv, int q_group, int has_kv, int dtype, dsb200_stream_t stream);
 /* out[t, h dv + c] = sum_j p_j v_j[c] over the keys j <= pos(t) of the token's sequence, p_j = exp(s_j) / (sink + sum_j exp(s_j)),
  * s_j = scale q_h . k_j, soft-capped as cap tanh(s_j / cap) when cap > 0.  q [T, q_ld] (H heads of d); query head h reads key/value head
  * h / (H / G); out [T, out_ld] (H heads of dv).  CUDA cores, fp32 scores and accumulation, any sizes; dtype 0 = bf16, 1 = fp32. */
@@ -607,7 +617,8 @@ int dsb200_sink_attention(const void* q, long long q_ld, const void* k_cache, lo
                           dsb200_stream_t stream);
 /* `sink_attention` with learned sinks, a distance term, a mask by parts and free strides:
  *   sink_logit [H] (or null): exp(sink_logit[h]) joins head h's denominator;   r1, r2 [H] (or both null): s_j -= r1[h] ln(1 + r2[h] (pos - j));
- *   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible;
+ *   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible; window > 0: only
+ *   the keys with pos - j < window;
  *   q[t * q_ld + h * q_head_stride + c], out[t * out_ld + h * out_head_stride + c]; a cached key / value head starts every k_row / v_row
  *   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start). */
 int dsb200_sink_attention_ex(const void* q, long long q_ld, long long q_head_stride, const void* k_cache,
@@ -615,7 +626,7 @@ int dsb200_sink_attention_ex(const void* q, long long q_ld, long long q_head_str
                              const int* tok_seq, const int* tok_pos, const int* block_table, int bt_stride, int block_size,
                              void* out, long long out_ld, long long out_head_stride, int n_tokens, int H, int G, int d,
                              int dv, float scale, float cap, float sink, const float* sink_logit, const float* r1,
-                             const float* r2, int part, int dtype, dsb200_stream_t stream);
+                             const float* r2, int part, int window, int dtype, dsb200_stream_t stream);
 /* Low-rank attention with one rotated key part shared by the heads.  proj [T, ld] (dtype 0 = bf16, 1 = fp32) holds per token the H query heads
  * (d plain entries, then dr entries to rotate) from q_col0 and the low-rank row (R entries, then dr entries to rotate) from kv_col0.  The
  * query heads' rotated parts are rotated IN PLACE (first rot_dims of the dr entries; entry i pairs with entry i + rot_dims / 2; angle =
@@ -639,6 +650,26 @@ int dsb200_conv_head_norm_append(const void* proj, long long ld, int col0, const
                                  long long v_block_stride, void* q_out, long long q_ld, const void* v_other,
                                  const float* mix, void* v_own, int n_tokens, int H, int G, int d, int dv, int taps,
                                  float eps, int q_row, int k_row, int v_row, int dtype, dsb200_stream_t stream);
+
+/* ---- csrc/ragged/ssd_ops.cu */
+/* proj [T, ld] (dtype 0 = bf16, 1 = fp32) holds per token C channels (x | B | C of the recurrence) from col0 and H step-size pre-activations
+ * from dt_col0.  xbc [T, C] = silu(b + sum_j w[j, :] u_(t - taps + 1 + j)) with w fp32 [taps, C], b fp32 [C]; rows before this step come from
+ * state [slots, taps - 1, C] (null when taps = 1), rows before the sequence are zeros.  dt [T, H] = softplus(pre + dt_bias), la [T, H] = -rate dt
+ * (fp32).  Update the state afterwards with dsb200_conv_state_update. */
+int dsb200_ssd_prepare(const void* proj, long long ld, int col0, int dt_col0, const float* w, const float* b,
+                       const void* state, const int* seq_desc, const int* tok_seq, const float* dt_bias, const float* rate,
+                       void* xbc, float* dt, float* la, int n_tokens, int C, int H, int taps, int dtype,
+                       dsb200_stream_t stream);
+/* The recurrence over every sequence's new tokens in order, for the sequences that bring min_new .. max_new tokens.  xbc [T, H P + 2 G N]
+ * (x | B | C, head h reads group h / (H / G)), dt and la fp32 [T, H] as dsb200_ssd_prepare leaves them, Dskip fp32 [H]; state fp32
+ * [slots, H, N, P]; out fp32 [T, H P].  Any sizes with N <= 512 (1024 when P is a multiple of 4). */
+int dsb200_ssd_scan(const void* xbc, const float* dt, const float* la, const float* Dskip, const int* seq_desc,
+                    float* state, float* out, int n_seqs, int H, int G, int N, int P, int min_new, int max_new, int dtype,
+                    dsb200_stream_t stream);
+/* out[t, :] = rms-in-groups(y[t, :] silu(z[t, :])) * w over `inner` values in `groups` equal consecutive parts (eps inside the root); y fp32
+ * [T, inner]; z [T, z_ld] and out [T, out_ld] in the activation dtype (0 = bf16, 1 = fp32), w fp32 [inner]. */
+int dsb200_gated_group_norm(const float* y, const void* z, long long z_ld, const float* w, void* out, long long out_ld,
+                            int n_tokens, int inner, int groups, float eps, int dtype, dsb200_stream_t stream);
 
 /* ---- csrc/random_ltd/token_ops.cu */
 /* idx: int32 [rows, reserved] of unique positions in [0, seq); sorted ascending in place, row by row. */
