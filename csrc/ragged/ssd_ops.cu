@@ -178,7 +178,11 @@ ssd_prepare_kernel(const T* __restrict__ proj, long long ld, int col0, int dt_co
 // thread (tx, ty) keeps rows ty, ty + TY, ... (RPT of them) of its V columns in registers.  Tokens are staged SCAN_CHUNK at a time; a thread
 // leaves its part of every token's read-out in shared memory and the block adds the TY parts after the chunk (no reduction per token).
 // The state in memory is [slots, H, N, P], so that a warp reads whole stretches of a row.
+//
+// A decay close to 1 is applied as S + (exp(la) - 1) S: the rounding of exp(la) itself would act on a slowly fading state in the same direction
+// thousands of times, that of expm1 is smaller by the factor 1 - exp(la).
 constexpr int SCAN_THREADS = 256, SCAN_CHUNK = 8;
+constexpr float SLOW_DECAY = -0.7f;
 template <typename T, int V, int RPT>
 __global__ void __launch_bounds__(SCAN_THREADS)
 ssd_scan_kernel(const T* __restrict__ xbc, const float* __restrict__ dt, const float* __restrict__ la, const float* __restrict__ Dskip,
@@ -223,7 +227,10 @@ ssd_scan_kernel(const T* __restrict__ xbc, const float* __restrict__ dt, const f
       const int tok = x / cols, p = x - tok * cols;
       xs[tok * PT + p] = to_f(xbc[static_cast<size_t>(sd.x + t0 + tok) * C + h * P + p0 + p]);
     }
-    if (tid < cn) es[tid] = expf(la[static_cast<size_t>(sd.x + t0 + tid) * H + h]);
+    if (tid < cn) {
+      const float l = la[static_cast<size_t>(sd.x + t0 + tid) * H + h];
+      es[tid] = l > SLOW_DECAY ? expm1f(l) : fmaxf(expf(l), 1e-38f);  // what the walk below multiplies by; the sign tells which
+    }
     __syncthreads();
     if (live) {
       for (int tok = 0; tok < cn; ++tok) {
@@ -239,7 +246,7 @@ ssd_scan_kernel(const T* __restrict__ xbc, const float* __restrict__ dt, const f
             const float bb = bs[tok * N + n], cc = cs[tok * N + n];
 #pragma unroll
             for (int k = 0; k < V; ++k) {
-              S[i][k] = fmaf(e, S[i][k], bb * xv[k]);
+              S[i][k] = fmaf(e, S[i][k], e > 0.f ? bb * xv[k] : fmaf(bb, xv[k], S[i][k]));
               acc[k] = fmaf(cc, S[i][k], acc[k]);
             }
           }

@@ -892,6 +892,7 @@ def conv_head_norm_append(proj, col0, bias, conv_w, wq, wk, state, seq_desc, tok
 native.register_sigs({
     "dsb200_ssd_prepare": "p l ii ppp pp pp ppp iiii i p",
     "dsb200_ssd_scan": "ppppp pp iiiii ii i p",
+    "dsb200_ssd_chunk": "ppppp ppp iiiiii i p",
     "dsb200_gated_group_norm": "pp l pp l iii f i p",
 })
 
@@ -925,6 +926,36 @@ def ssd_scan(xbc, dt, la, D, seq_desc, n_seqs, state, H, G, N, P, out=None, min_
         out = torch.empty(T, H * P, dtype=torch.float32, device=xbc.device)
     native.check(native.lib().dsb200_ssd_scan(native.ptr(xbc), native.ptr(dt), native.ptr(la), native.ptr(D), native.ptr(seq_desc), native.ptr(state),
                                               native.ptr(out), n_seqs, H, G, N, P, int(min_new), int(max_new), _dt(xbc), native.stream_ptr()))
+    return out
+
+
+_wait_errors = {}
+
+
+def wait_error_word(device):
+    """One int32 per device that kernels with bounded waits set to 1 when a wait gave up (their outputs are then incomplete)."""
+    if device not in _wait_errors:
+        _wait_errors[device] = torch.zeros(1, dtype=torch.int32, device=device)
+    return _wait_errors[device]
+
+
+def ssd_chunk_ok(xbc, H, G, N, P):
+    """Whether the tensor-core form of the recurrence takes these sizes: bf16, state rows a multiple of 16 up to 128, columns a multiple of 16 up
+    to 64, at least 64 channels."""
+    return (xbc.is_cuda and xbc.dtype == torch.bfloat16 and xbc.is_contiguous() and xbc.data_ptr() % 16 == 0 and N % 16 == 0 and 16 <= N <= 128 and
+            P % 16 == 0 and 16 <= P <= 64 and H * P + 2 * G * N >= 64 and os.environ.get("DSB200_SSD_CHUNK", "1") != "0")
+
+
+def ssd_chunk(xbc, dt, la, D, seq_desc, n_seqs, state, out, H, G, N, P, min_new=1):
+    """`ssd_scan` in its chunked form on the tensor cores (csrc/ragged/ssd_chunk.cu), for the sequences that bring at least `min_new` tokens."""
+    T = xbc.shape[0]
+    assert ssd_chunk_ok(xbc, H, G, N, P) and xbc.shape[1] == H * P + 2 * G * N and D.dtype == torch.float32 and D.numel() == H
+    assert all(t.dtype == torch.float32 and t.is_contiguous() and t.shape == (T, H) for t in (dt, la))
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, N, P)
+    assert out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (T, H * P)
+    native.check(native.lib().dsb200_ssd_chunk(native.ptr(xbc), native.ptr(dt), native.ptr(la), native.ptr(D), native.ptr(seq_desc), native.ptr(state),
+                                               native.ptr(out), native.ptr(wait_error_word(xbc.device)), T, n_seqs, H, G, N, P, int(min_new),
+                                               native.stream_ptr()))
     return out
 
 

@@ -4,7 +4,9 @@ Per layer and step, from the fused projection: `ssd_prepare` (convolution with b
 `conv_state_update` (the last taps - 1 rows become the sequence's state), the recurrence, and `gated_group_norm` (times silu(z), RMS norm in
 equal parts, weight).  csrc/ragged/ssd_ops.cu.
 
-The recurrence is `ssd_scan`: token by token with the state in registers, any sizes, fp32 arithmetic for both activation dtypes.  The state of a
+Two forms of the recurrence.  `ssd_scan`: token by token with the state in registers, any sizes, fp32 arithmetic for both activation dtypes --
+decode steps, short portions, fp32.  `ssd_chunk` (csrc/ragged/ssd_chunk.cu): chunks of 128 tokens as matrix products on the tensor cores, bf16
+with state rows up to 128 and columns up to 64 -- the sequences of a step that bring at least CHUNK_MIN tokens.  The state of a
 head lives in the state manager's slots as fp32 [state_size, value_size] and starts at zero (a sequence at position 0 ignores what its slot
 held)."""
 from typing import Any, Dict, List, Type
@@ -17,6 +19,8 @@ from ....inference_utils import DtypeEnum
 from ....ragged.state_slots import StateBufferSpec
 from ...configs import DSStateSpaceConfig
 from ...interfaces import DSRecurrentMixerBase, DSRecurrentRegistry
+
+CHUNK_MIN = 32  # new tokens of a sequence from which on the chunked form is the faster one
 
 
 @DSRecurrentRegistry.register_module
@@ -82,5 +86,12 @@ class DSStateSpace(DSRecurrentMixerBase):
         xbc, dt, la = K.ssd_prepare(proj, x0, x0 + C, conv_w, conv_b, conv_state, desc, batch.tok_seq(), dt_bias, rate, C, H, c.conv_taps)
         if conv_state is not None:
             K.conv_state_update(proj, x0, C, conv_state, 0, desc, n_seqs, c.conv_taps)
-        y = K.ssd_scan(xbc, dt, la, skip, desc, n_seqs, state_manager.get_state(prefix + ".S"), H, G, N, P)
+        state = state_manager.get_state(prefix + ".S")
+        y = torch.empty(proj.shape[0], self.inner, dtype=torch.float32, device=proj.device)
+        longest, shortest = batch.portion_range
+        chunked = longest >= CHUNK_MIN and K.ssd_chunk_ok(xbc, H, G, N, P)
+        if chunked:
+            K.ssd_chunk(xbc, dt, la, skip, desc, n_seqs, state, y, H, G, N, P, min_new=CHUNK_MIN)
+        if not chunked or shortest < CHUNK_MIN:
+            K.ssd_scan(xbc, dt, la, skip, desc, n_seqs, state, H, G, N, P, out=y, **({"max_new": CHUNK_MIN - 1} if chunked else {}))
         return K.gated_group_norm(y, proj[:, col0:col0 + self.inner], norm_w, out, c.norm_groups, c.eps)

@@ -161,6 +161,11 @@ class RaggedBatchWrapper:
         return self._n_seqs
 
     @property
+    def portion_range(self):
+        """(most, fewest) new tokens a sequence of the batch brings; known on the host, so that launches can be chosen by it."""
+        return (max(self._seq_ntok), min(self._seq_ntok)) if self._seq_ntok else (0, 0)
+
+    @property
     def is_pure_prefill(self):
         """every sequence of the batch is new (no KV history) -- the dense flash kernel can be used per sequence"""
         return all(s == 0 for s in self._seq_seen)

@@ -651,6 +651,15 @@ int dsb200_conv_head_norm_append(const void* proj, long long ld, int col0, const
                                  const float* mix, void* v_own, int n_tokens, int H, int G, int d, int dv, int taps,
                                  float eps, int q_row, int k_row, int v_row, int dtype, dsb200_stream_t stream);
 
+/* ---- csrc/ragged/ssd_chunk.cu */
+/* The recurrence of dsb200_ssd_scan in its chunked form, for the sequences that bring at least min_new tokens (the others are left to
+ * dsb200_ssd_scan with max_new = min_new - 1).  xbc bf16 [T, H P + 2 G N], the rest as there; N a multiple of 16 up to 128, P a multiple of 16 up
+ * to 64, at least 64 channels, rows 16-byte aligned.  error: one int on the device, set to 1 when a wait inside the kernel gave up (the outputs are
+ * then incomplete); never cleared. */
+int dsb200_ssd_chunk(const void* xbc, const float* dt, const float* la, const float* Dskip, const int* seq_desc,
+                     float* state, float* out, int* error, int n_tokens, int n_seqs, int H, int G, int N, int P,
+                     int min_new, dsb200_stream_t stream);
+
 /* ---- csrc/ragged/ssd_ops.cu */
 /* proj [T, ld] (dtype 0 = bf16, 1 = fp32) holds per token C channels (x | B | C of the recurrence) from col0 and H step-size pre-activations
  * from dt_col0.  xbc [T, C] = silu(b + sum_j w[j, :] u_(t - taps + 1 + j)) with w fp32 [taps, C], b fp32 [C]; rows before this step come from
