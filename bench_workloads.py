@@ -1236,4 +1236,243 @@ def run_midulorn(args):
           flush=True)
 
 
-WORKLOADS = {"fastgen70b": run_fastgen70b, "mixtral": run_mixtral, "ulysses13b": run_ulysses13b, "linasun": run_linasun, "kulanex": run_kulanex, "pudinex": run_pudinex, "midulorn": run_midulorn}
+# ---------------------------------------------------------------------------------------------------------------- Gepolix
+GEPOLIX_SIZES = PUDINEX_SIZES  # the same widths, heads, experts and vocabularies: the twins are built from one tuple
+GEPOLIX_WINDOW, GEPOLIX_TAPS, GEPOLIX_STATE, GEPOLIX_VDIM, GEPOLIX_GROUPS = 1024, 4, 128, 64, 8
+
+
+def _gepolix_state(torch, dev, W, L, H, d, hkv, E, top, ff, V):
+    """Layers alternate 'mamba2' (inner width 2 W in heads of 64, 128 x 64 states, 8 groups, 4 taps) and 'attention' (H:hkv heads of d, every entry
+    rotated, window 1024; every second one reads the cache of the one before), all with the MoE feed-forward (a gated shared expert of the
+    experts' size)."""
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": E, "top": top}, "shared": {"ff": ff}}
+    inner = 2 * W
+    ssm = {"heads": inner // GEPOLIX_VDIM, "vdim": GEPOLIX_VDIM, "state": GEPOLIX_STATE, "groups": GEPOLIX_GROUPS, "conv": GEPOLIX_TAPS, "norm_groups": GEPOLIX_GROUPS}
+    att = {"heads": H, "kv_heads": hkv, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": GEPOLIX_WINDOW}, "rot": {"base": 1e6, "dims": d}}
+    layers, owner = [], None
+    for i in range(L):
+        if i % 2 == 0:
+            layers.append({"type": "mamba2", "mixer": ssm, "mlp": moe})
+        else:
+            layers.append({"type": "attention", "mixer": att if owner is None else dict(att, kv_from=owner), "mlp": moe})
+            owner = i if owner is None else None
+    cfg = {"architecture": "Gepolix", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "layers": layers}
+
+    def r(*shape, std=0.02, mean=0.0):
+        return torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(mean, std)
+
+    def norm(name):
+        return {name: r(W, mean=1.0), name + ".b": r(W), name + ".alpha": torch.full((), 0.5, device=dev, dtype=torch.bfloat16)}
+
+    sd = {"embed": r(V, W, std=1.0), "head": r(V, W), **norm("final.norm")}
+    nh, C = ssm["heads"], inner + 2 * GEPOLIX_GROUPS * GEPOLIX_STATE
+    for i, Lc in enumerate(layers):
+        p, a = f"l{i}.", f"l{i}.mix."
+        sd.update(norm(p + "norm1"))
+        sd.update({p + "mlp.router": r(E, W, std=0.5), p + "mlp.router.b": r(E), p + "mlp.shared.gate": r(ff, W), p + "mlp.shared.up": r(ff, W),
+                   p + "mlp.shared.down": r(W, ff), p + "mlp.shared.sg": r(1, W)})
+        for e in range(E):
+            sd.update({p + f"mlp.e{e}.gate": r(ff, W), p + f"mlp.e{e}.up": r(ff, W), p + f"mlp.e{e}.down": r(W, ff)})
+        if Lc["type"] == "mamba2":
+            sd.update({a + "in": r(inner + C + nh, W), a + "conv": r(C, GEPOLIX_TAPS, std=0.5), a + "conv.b": r(C), a + "dt_bias": r(nh, mean=-2.0, std=1.0),
+                       a + "A_log": r(nh, std=1.0), a + "D": r(nh, mean=1.0), a + "norm": r(inner, mean=1.0), a + "o": r(W, inner)})
+        else:
+            sd.update({a + "q": r(H * d, W), a + "q.b": r(H * d), a + "o": r(W, H * d)})
+            if "kv_from" not in Lc["mixer"]:
+                sd.update({a + "k": r(hkv * d, W), a + "k.b": r(hkv * d), a + "v": r(hkv * d, W), a + "v.b": r(hkv * d)})
+    return cfg, sd
+
+
+def _gepolix_kernel_table(torch, peaks, W, H, d, hkv, E, top, ff, T, ctx, n_dec):
+    """Every kernel of the design beside the like kernel of the closest family (Pudinex; Midulorn for the convolution, Kulanex for the window),
+    isolated, with the fraction of the measured roofline (HBM copy bandwidth for the streaming kernels, cuBLAS bf16 rate for attention prefill)."""
+    from deepspeedsyclsupport_b200.inference.v2 import kernels as K
+    from deepspeedsyclsupport_b200.inference.v2.modules.configs import RampRotaryScalingConfig
+    from deepspeedsyclsupport_b200.inference.v2.modules.implementations.attention.sink_blocked_attention import ramp_scaled_frequencies
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, ms, like, like_ms, nbytes=None, like_bytes=None, flops=None, like_flops=None):
+        def frac(ms_, b, f):
+            return round(max((b or 0) / hbm, (f or 0) / tf) / (ms_ * 1e-3), 4)
+        rows.append({"kernel": name, "ms": round(ms, 4), "roofline_frac": frac(ms, nbytes, flops), "like": like, "like_ms": round(like_ms, 4),
+                     "like_roofline_frac": frac(like_ms, like_bytes if like_bytes is not None else nbytes, like_flops if like_flops is not None else flops)})
+
+    def rnd(*shape):
+        return torch.randn(*shape, device=dev)
+
+    def ms(f, n=20):
+        return _event_ms(torch, f, n, flush)
+
+    x32, y, y32, g32, al = rnd(T, W), rnd(T, W).to(bf), rnd(T, W), rnd(W), torch.full((1, ), 0.5, device=dev)
+    add("stream_tanh_norm (bf16 + fp32 branch in, bf16 + fp32 copy out)", ms(lambda: K.stream_tanh_norm(x32, (y, ), y32, al, g32, g32, fp32_copy=True)),
+        "stream_group_norm (2 parts; same branches and copies; Pudinex)", ms(lambda: K.stream_group_norm(x32, (y, ), y32, g32, 2, 1e-6, fp32_copy=True)),
+        nbytes=T * W * (4 + 2 + 4 + 4 + 2 + 4))
+    lg, rb = rnd(T, E), rnd(E)
+    add("grouped_topk_gating (biased logits, softmax over the chosen)", ms(lambda: K.grouped_topk_gating(lg, top, normalize=True, bias=rb)),
+        "grouped_topk_gating (softmax, correction, renormalised; Pudinex)", ms(lambda: K.grouped_topk_gating(lg, top, rb, normalize=True)), nbytes=T * (E * 4 + top * 12))
+    gu, act = rnd(T, 2 * ff + 8).to(bf), torch.empty(T, ff, device=dev, dtype=bf)
+    add("clamped_swish_gate_cols, one gate per token on top", ms(lambda: K.clamped_swish_gate_cols(gu, 0, ff, ff, act, 1.0, float("inf"), 0.0, row_gate_col=2 * ff)),
+        "clamped_swish_gate_cols (Pudinex)", ms(lambda: K.clamped_swish_gate_cols(gu, 0, ff, ff, act, 1.0, float("inf"), 0.0)), nbytes=T * ff * 6)
+    bs, inner, N, P, G = 128, 2 * W, GEPOLIX_STATE, GEPOLIX_VDIM, GEPOLIX_GROUPS
+    nh, C = inner // P, inner + 2 * G * N
+    freq = ramp_scaled_frequencies(d, 1e6)[0].to(dev)
+    pfreq, pmag = ramp_scaled_frequencies(d // 2, 1e6, RampRotaryScalingConfig(factor=8.0, original=8192, fast=32.0, slow=1.0))
+    pfreq = pfreq.to(dev)
+    for label, n_seq, new, seen in (("prefill", max(1, T // 2048), min(T, 2048), ctx), ("decode", n_dec, 1, ctx)):
+        per = -(-(seen + new) // bs)
+        nb, Tn, dec = n_seq * per, n_seq * new, label == "decode"
+        bt = torch.arange(nb, dtype=torch.int32, device=dev).view(n_seq, per)
+        tok_seq = torch.arange(n_seq, dtype=torch.int32, device=dev).repeat_interleave(new)
+        tok_pos = (seen + torch.arange(new, dtype=torch.int32, device=dev)).repeat(n_seq)
+        desc = torch.tensor([[i * new, new, seen, i] for i in range(n_seq)], dtype=torch.int32, device=dev)
+        kv, qkv = rnd(nb, 2, bs, hkv, d).to(bf), rnd(Tn, (H + 2 * hkv) * d).to(bf)
+        nw, qo = rnd(d), torch.empty(Tn, H * d, device=dev, dtype=bf)
+        bq, bk = rnd(H * d), rnd(hkv * d)
+        planes = K.cache_planes(kv)
+
+        def append(biases, kv_part, w, f, mag, rot, norm_v):
+            return lambda: K.head_norm_rotary_append(qkv, 0, H * d, (H + hkv) * d, w, w, f, mag, tok_seq, tok_pos, bt, bs, planes[0], planes[1], qo, H, hkv, d, d,
+                                                     rot, 1e-6, norm_v=norm_v, biases=biases, kv=kv_part)
+        like = ms(append(None, True, nw, pfreq, pmag, d // 2, True), 10)
+        C_att = (H + 2 * hkv) * d
+        add(f"head_norm_rotary_append, biases instead of norms, every entry rotated, {label}", ms(append((bq, bk, bk), True, None, freq, 1.0, d, False), 10),
+            f"head_norm_rotary_append (Pudinex: norms, half rotated), {label}", like, nbytes=Tn * C_att * 4)
+        add(f"head_norm_rotary_append, queries only, {label}", ms(append((bq, None, None), False, None, freq, 1.0, d, False), 10),
+            f"head_norm_rotary_append (Pudinex: norms, half rotated), {label}", like, nbytes=Tn * H * d * 4, like_bytes=Tn * C_att * 4)
+        out = torch.empty(Tn, H * d, device=dev, dtype=bf)
+        wk = n_seq * sum(min(p + 1, GEPOLIX_WINDOW) for p in range(seen, seen + new))
+        abytes = n_seq * min(seen + new, GEPOLIX_WINDOW + new) * hkv * d * 4 + Tn * H * d * 4
+        add(f"attention, window {GEPOLIX_WINDOW}, tcgen05, {label} (GQA {H}:{hkv})",
+            ms(lambda: K.paged_flash_sink(qo, kv, tok_seq, tok_pos, bt, out, H, hkv, d, d ** -0.5, 0.0, 0.0, window=GEPOLIX_WINDOW, decode=dec), 10),
+            f"windowed attention with 4 kept keys, tcgen05, {label} (Kulanex)",
+            ms(lambda: K.paged_flash_window(qo, kv, tok_seq, tok_pos, bt, out, H, hkv, d, GEPOLIX_WINDOW, 4, d ** -0.5, decode=dec), 10), nbytes=abytes, flops=4.0 * wk * H * d)
+        # state-space mixer
+        proj = rnd(Tn, inner + C + nh).to(bf)
+        cw, cb, db, rate, D, nrm = rnd(GEPOLIX_TAPS, C), rnd(C), rnd(nh) - 2, rnd(nh).exp(), rnd(nh), rnd(inner)
+        cstate = torch.zeros(n_seq, GEPOLIX_TAPS - 1, C, device=dev, dtype=bf)
+
+        def prep():
+            K.conv_state_update(proj, inner, C, cstate, 0, desc, n_seq, GEPOLIX_TAPS)
+            return K.ssd_prepare(proj, inner, inner + C, cw, cb, cstate, desc, tok_seq, db, rate, C, nh, GEPOLIX_TAPS)
+        C2 = (H + 2 * hkv) * d
+        cw2, cb2, mix = rnd(GEPOLIX_TAPS, C2), rnd(C2), torch.full((1, ), 0.3, device=dev)
+        cs2, vsrc = torch.zeros(n_seq, GEPOLIX_TAPS - 1, C2, device=dev, dtype=bf), rnd(Tn, hkv * d).to(bf)
+
+        def cprep():
+            K.conv_head_norm_append(qkv, 0, cb2, cw2, nw, nw, cs2, desc, tok_seq, tok_pos, bt, bs, planes[0], planes[1], qo, H, hkv, d, d, GEPOLIX_TAPS, 1e-6,
+                                    v_other=vsrc, mix=mix)
+            K.conv_state_update(qkv, 0, C2, cs2, 0, desc, n_seq, GEPOLIX_TAPS)
+        add(f"ssd_prepare + conv_state_update ({C} channels, {GEPOLIX_TAPS} taps), {label}", ms(prep, 10),
+            f"conv_head_norm_append + conv_state_update ({C2} channels; Midulorn), {label}", ms(cprep, 10), nbytes=Tn * (C * 4 + nh * 10),
+            like_bytes=Tn * (C2 * 4 + hkv * d * 2))
+        xbc, dt, la = prep()
+        S = torch.zeros(n_seq, nh, N, P, device=dev)
+        yo = torch.empty(Tn, inner, device=dev)
+        tproj = rnd(Tn, 3 * H * d).to(bf)
+        fb, lo = torch.full((H * d, ), 2.0, device=dev), torch.full((H * d, ), 0.5, device=dev)
+        tS = torch.zeros(n_seq, H, K.scan_state_floats(d, d), device=dev)
+        like = ms(lambda: K.tied_gate_scan(tproj, 0, H * d, 2 * H * d, fb, lo, desc, n_seq, tS, H, d, d), 5)
+        sbytes, lbytes = Tn * (C * 2 + nh * 8 + inner * 4) + n_seq * nh * N * P * 8, Tn * H * d * (3 * 2 + 4) + n_seq * H * d * d * 8
+        like_name = f"tied_gate_scan ({H} x {d} x {d}; Pudinex), {label}"
+        if not dec:
+            add(f"ssd_chunk ({nh} x {N} x {P}), {label}", ms(lambda: K.ssd_chunk(xbc, dt, la, D, desc, n_seq, S, yo, nh, G, N, P), 10), like_name, like,
+                nbytes=sbytes, like_bytes=lbytes)
+        add(f"ssd_scan ({nh} x {N} x {P}), {label}" + ("" if dec else " (not the path taken)"),
+            ms(lambda: K.ssd_scan(xbc, dt, la, D, desc, n_seq, S, nh, G, N, P, out=yo), 5), like_name, like, nbytes=sbytes, like_bytes=lbytes)
+        og, o2 = torch.empty(Tn, inner, device=dev, dtype=bf), rnd(Tn, H * d)
+        oh = torch.empty(Tn, H * d, device=dev, dtype=bf)
+        add(f"gated_group_norm ({inner} in {GEPOLIX_GROUPS} parts), {label}", ms(lambda: K.gated_group_norm(yo, proj[:, :inner], nrm, og, GEPOLIX_GROUPS, 1e-6), 10),
+            f"head_norm_gate without a gate ({H * d}; Pudinex), {label}", ms(lambda: K.head_norm_gate(o2, nw, None, oh, H, d, 1e-6, shared_weight=True), 10),
+            nbytes=Tn * inner * 8, like_bytes=Tn * H * d * 6)
+    return rows
+
+
+def run_gepolix(args):
+    """Prefill and decode throughput of Gepolix through the FastGen engine at a few layer sizes, beside a Pudinex (the closest family: layers whose
+    sublayers share one norm, matrix states in the state slots, softmax router, shared expert) and a Mixtral of equal size (same width,
+    layers, heads, experts, ff, top-k, vocabulary), plus the isolated kernels of the design beside their likes."""
+    sys.path.insert(0, ROOT)
+    import torch
+    import deepspeedsyclsupport_b200 as deepspeed
+    from deepspeedsyclsupport_b200 import comm as dist
+    from deepspeedsyclsupport_b200.inference.v2 import RaggedInferenceEngineConfig, build_engine_from_state_dict
+    from deepspeedsyclsupport_b200.ops import native
+    deepspeed.init_distributed()
+    assert dist.get_world_size() == 1, "--workload gepolix is a one-GPU comparison"
+    dev = torch.device("cuda", torch.cuda.current_device())
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+        peaks = dict(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))), source="measured")
+    n_seqs, prompt, budget = min(args.sequences, 64), 1024, 4096
+    results, clocks, l0 = {}, None, native.launch_count
+    g = torch.Generator().manual_seed(11)
+    for name in (args.model.split(",") if args.model != "7b" else ["s", "m"]):
+        W, L, H, d, hkv, E, top, ff, V = GEPOLIX_SIZES[name]
+        max_ctx = -(-(prompt + 4 * (args.steps + args.warmup) * 4 + 64) // 128) * 128
+        ecfg = RaggedInferenceEngineConfig(state_manager={"max_ragged_batch_size": budget, "max_ragged_sequence_count": n_seqs, "max_tracked_sequences": n_seqs,
+                                                          "max_context": max_ctx, "memory_config": {"mode": "allocate", "size": n_seqs * (max_ctx // 128) + 4}})
+        res = {}
+        for fam in ("gepolix", "pudinex", "mixtral"):
+            if fam == "gepolix":
+                cfg, sd = _gepolix_state(torch, dev, W, L, H, d, hkv, E, top, ff, V)
+            elif fam == "pudinex":
+                cfg, sd = _pudinex_state(torch, dev, W, L, H, d, hkv, E, top, ff, V)
+            else:
+                cfg, sd = _mixtral_state(torch, dev, W, L, H, d, hkv, E, top, ff, V)
+            eng = build_engine_from_state_dict(fam, cfg, sd, ecfg, dtype=torch.bfloat16)
+            n_params = sum(v.numel() for v in sd.values())
+            del sd
+            prompts = [torch.randint(0, V, (prompt, ), generator=g).pin_memory() for _ in range(n_seqs)]
+            uids = list(range(n_seqs))
+            state = {"live": False, "next": None}
+
+            def prefill():
+                if state["live"]:
+                    for u in uids:
+                        eng.flush(u)
+                per = budget // prompt
+                nxt = torch.zeros(n_seqs, dtype=torch.long)
+                for i in range(0, n_seqs, per):
+                    us = uids[i:i + per]
+                    nxt[i:i + len(us)] = eng.put(us, [prompts[u] for u in us]).argmax(-1).cpu()
+                state["live"], state["next"] = True, nxt
+
+            def decode():
+                nxt = state["next"]
+                for _ in range(4):
+                    nxt = eng.put(uids, [nxt[u:u + 1] for u in uids]).argmax(-1).cpu()
+                state["next"] = nxt
+
+            ms_p, _ = _timed(torch, dist, prefill, args.steps, 3)
+            ms_d, clk = _timed(torch, dist, decode, args.steps, args.warmup)
+            if fam == "gepolix":
+                clocks = clk
+            res[fam] = {"params_b": round(n_params / 1e9, 3), "prefill_tokens_per_s": round(n_seqs * prompt / ms_p * 1e3, 1), "prefill_ms": round(ms_p, 2),
+                        "decode_tokens_per_s": round(n_seqs * 4 / ms_d * 1e3, 1), "decode_ms_per_step": round(ms_d / 4, 3)}
+            del eng
+            torch.cuda.empty_cache()
+        for other in ("pudinex", "mixtral"):
+            res["gepolix_over_" + other] = {"prefill": round(res["gepolix"]["prefill_tokens_per_s"] / res[other]["prefill_tokens_per_s"], 3),
+                                             "decode": round(res["gepolix"]["decode_tokens_per_s"] / res[other]["decode_tokens_per_s"], 3)}
+        res["shape"] = {"width": W, "layers": L, "heads": H, "head_dim": d, "kv_heads": hkv, "experts": E, "top": top, "ff": ff, "window": GEPOLIX_WINDOW,
+                        "taps": GEPOLIX_TAPS, "state": [GEPOLIX_STATE, GEPOLIX_VDIM], "inner": 2 * W}
+        res["kernels"] = _gepolix_kernel_table(torch, peaks, W, H, d, hkv, E, top, ff, 4096, 2048, n_seqs)
+        results[name] = res
+    launches = native.launch_count - l0
+    last = results[list(results)[-1]]
+    extra = {"results": results, "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops", "source")},
+             "e2e": {"value": last["gepolix"]["decode_tokens_per_s"], "unit": "generated tokens/s", "h2d_bytes_per_step": n_seqs * 8, "d2h_bytes_per_step": n_seqs * 8},
+             "reference_arm": "none: the reference has no model of this design"}
+    config = {"model": "gepolix (random weights) beside pudinex and mixtral of equal size", "sizes": list(results), "sequences": n_seqs, "prompt_len": prompt,
+              "token_budget_per_forward": budget, "decode_steps_per_timed_step": 4, "kv_block": 128,
+              "l2_policy": "engine steps: weights exceed the 126 MB L2, no flush; isolated kernels: 256 MB write before every timed run"}
+    print(json.dumps(_line("generated tokens/sec Gepolix FastGen ragged decode, 1 GPU (prefill, a Pudinex and a Mixtral of equal size alongside)",
+                           last["gepolix"]["decode_tokens_per_s"], "tokens/s", 1, args, last["gepolix"]["decode_ms_per_step"], config, clocks, launches, extra)),
+          flush=True)
+
+
+WORKLOADS = {"fastgen70b": run_fastgen70b, "mixtral": run_mixtral, "ulysses13b": run_ulysses13b, "linasun": run_linasun, "kulanex": run_kulanex, "pudinex": run_pudinex, "midulorn": run_midulorn,
+             "gepolix": run_gepolix}

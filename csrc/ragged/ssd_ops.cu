@@ -80,7 +80,7 @@ __device__ __forceinline__ float silu_t(float z) {
 __device__ __forceinline__ float softplusf_(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 // ------------------------------------------------------------------------------------------------------------------ prepare
-// A thread owns V channels and walks PREP_ROWS consecutive rows of the batch; the taps - 1 rows in front of the current one stay in
+// A thread owns V channels and walks `rows` consecutive rows of the batch (PREP_ROWS of them; one when there are few rows: decode steps); the taps - 1 rows in front of the current one stay in
 // registers (TAPS > 0; TAPS = 0: any number of taps, every row read per tap).  When the walk enters another sequence -- or starts in the
 // middle of one -- that window is filled from the rows of this step, the state, or zeros.
 constexpr int PREP_ROWS = 8, PREP_THREADS = 128;
@@ -89,8 +89,8 @@ __global__ void __launch_bounds__(PREP_THREADS)
 ssd_prepare_kernel(const T* __restrict__ proj, long long ld, int col0, int dt_col0, const float* __restrict__ w, const float* __restrict__ b,
                    const T* __restrict__ state, const int4* __restrict__ seq_desc, const int* __restrict__ tok_seq, const float* __restrict__ dt_bias,
                    const float* __restrict__ rate, T* __restrict__ xbc, float* __restrict__ dt, float* __restrict__ la, int n_tokens, int C, int H,
-                   int taps, int conv_blocks) {
-  const int t_begin = blockIdx.y * PREP_ROWS, t_end = min(n_tokens, t_begin + PREP_ROWS);
+                   int taps, int conv_blocks, int rows) {
+  const int t_begin = blockIdx.y * rows, t_end = min(n_tokens, t_begin + rows);
   if (static_cast<int>(blockIdx.x) >= conv_blocks) {  // the step sizes: one thread per (row, head)
     for (int i = (blockIdx.x - conv_blocks) * PREP_THREADS + threadIdx.x; i < (t_end - t_begin) * H; i += (gridDim.x - conv_blocks) * PREP_THREADS) {
       const int t = t_begin + i / H, h = i % H;
@@ -354,11 +354,12 @@ DSB_EXPORT int dsb200_ssd_prepare(const void* proj, long long ld, int col0, int 
   DSB_REQUIRE(C >= 1 && H >= 1 && taps >= 1 && (taps == 1 || state != nullptr), "ssd_prepare: %d channels, %d heads, %d taps", C, H, taps);
   const bool vec = mult4(C) && mult4(ld) && mult4(col0) && al16(proj) && al16(w) && al16(b) && al16(state) && al16(xbc);
   const int V = vec ? 4 : 1;
-  const int conv_blocks = (C / V + PREP_THREADS - 1) / PREP_THREADS, dt_blocks = (H * PREP_ROWS + PREP_THREADS - 1) / PREP_THREADS;
-  const dim3 grid(conv_blocks + (dt_blocks < 4 ? dt_blocks : 4), (n_tokens + PREP_ROWS - 1) / PREP_ROWS);
+  const int rows = n_tokens <= 512 ? 1 : PREP_ROWS;
+  const int conv_blocks = (C / V + PREP_THREADS - 1) / PREP_THREADS, dt_blocks = (H * rows + PREP_THREADS - 1) / PREP_THREADS;
+  const dim3 grid(conv_blocks + (dt_blocks < 4 ? dt_blocks : 4), (n_tokens + rows - 1) / rows);
 #define LAUNCH(T, VV, TT)                                                                                                                              \
   ssd_prepare_kernel<T, VV, TT><<<grid, PREP_THREADS, 0, stream>>>((const T*)proj, ld, col0, dt_col0, w, b, (const T*)state, (const int4*)seq_desc, tok_seq, \
-                                                                   dt_bias, rate, (T*)xbc, dt, la, n_tokens, C, H, taps, conv_blocks)
+                                                                   dt_bias, rate, (T*)xbc, dt, la, n_tokens, C, H, taps, conv_blocks, rows)
 #define BY_TAPS(T, VV)                       \
   do {                                       \
     if (taps == 2) LAUNCH(T, VV, 2);         \

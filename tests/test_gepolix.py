@@ -433,6 +433,37 @@ def test_state_space_sequences_side_by_side_and_a_slot_taken_over(dt):
         assert at[u] == hs[u].shape[0] and _rel(torch.cat(got[u]), want[u]) < (2e-5 if dt == torch.float32 else 2e-2), u
 
 
+@gpu
+@pytest.mark.parametrize("dt", DTYPES)
+@pytest.mark.parametrize("taps,C,H", [(4, 48, 6), (3, 21, 2), (1, 16, 3), (7, 40, 5)])
+def test_convolution_and_steps_of_many_rows(taps, C, H, dt):
+    """More than 512 rows (several rows per thread): sequences of 1, 2, 300, 3 and 290 rows side by side, some new, some with kept rows, so that a
+    thread's run of rows enters new sequences in its middle."""
+    K = _K()
+    g = torch.Generator().manual_seed(taps)
+    seqs = [(1, 0), (2, 9), (300, 1), (3, 0), (290, 2), (1, 50)]  # (new rows, rows seen before)
+    total = sum(n for n, _ in seqs)
+    proj = torch.randn(total, 5 + C + H + 2, generator=g).to(dt)
+    w, b = torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
+    bias, rate = torch.randn(H, generator=g) * 3, torch.rand(H, generator=g) * 4
+    kept = torch.randn(len(seqs), max(taps - 1, 1), C, generator=g).to(dt)
+    want, at, desc, tok_seq = [], 0, [], []
+    for i, (n, seen) in enumerate(seqs):
+        tail = kept[i, :taps - 1].double().clone()
+        if seen < taps - 1:
+            tail[:taps - 1 - seen] = 0  # positions before the sequence's start: whatever the slot holds does not count
+        want.append(O.causal_conv_silu(proj[at:at + n, 5:5 + C].double(), w, b, tail)[0])
+        desc.append([at, n, seen, i])
+        tok_seq += [i] * n
+        at += n
+    desc, tok_seq = torch.tensor(desc, dtype=torch.int32).cuda(), torch.tensor(tok_seq, dtype=torch.int32).cuda()
+    state = kept.cuda() if taps > 1 else None
+    xbc, dt_, la = K.ssd_prepare(proj.cuda(), 5, 5 + C, w.t().contiguous().cuda(), b.cuda(), state, desc, tok_seq, bias.cuda(), rate.cuda(), C, H, taps)
+    assert _rel(xbc, torch.cat(want)) < (1e-6 if dt == torch.float32 else 5e-3)
+    step = torch.nn.functional.softplus(proj[:, 5 + C:5 + C + H].double() + bias.double(), threshold=1e9)
+    assert _rel(dt_, step) < 1e-6 and _rel(la, -rate.double() * step) < 1e-6
+
+
 def _recurrence_inputs(T, H, G, N, P, dt_range, rate, seed, dt):
     g = torch.Generator().manual_seed(seed)
     xbc = torch.randn(T, H * P + 2 * G * N, generator=g).to(dt)
