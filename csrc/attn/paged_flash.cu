@@ -80,10 +80,50 @@ struct Params {
   // distance term: the score of key j for the query at position i loses r1[head] ln(1 + r2[head] (i - j)), formed in the exp2 domain as
   // r1 log2(1 + r2 (i - j)) (one MUFU lg2 per score); nullptr = none.  Not combined with ALiBi or the soft cap.
   const float* r1;
-  const float* r2;
+  const float* r2;     // nullptr with r1 given: the linear term, the score loses r1[head] (i - j)
+  // compact output: heads leave without padding -- head_real * out_dv + c for c < out_dv, head_real = kvh * out_per + slot for slot < out_per (the
+  // other slots of a group have no head) -- and are multiplied by sigmoid(gate[t * gate_ld + head_real * out_dv + c]) when a gate is given.
+  // out_dv = 0: every slot leaves as D entries, no gate.
+  int out_dv, out_per;
+  int out_vec;         // gate and output rows allow 16-byte accesses (out_dv a multiple of 8)
+  const __nv_bfloat16* gate;
+  long long gate_ld;
   int part;            // > 0: a query at position i sees only the keys j <= i with j / part == i / part (parts counted from position 0)
   long long* trace;  // diagnostics only (DSB200_PF_TRACE=1): clock64 stamps of the first CTA with >= 8 pages, [page][8 events]
 };
+__device__ __forceinline__ float sigmoid_fast(float g) { return __fdividef(1.f, 1.f + ex2_fast(-1.4426950408889634f * g)); }
+// N consecutive entries o[0 .. N) (from column c of the head in slot `slot` of key / value head kvh, token t) to a compact output row
+template <int N>
+__device__ __forceinline__ void store_compact(const Params& p, int t, int kvh, int slot, int c, const float* o) {
+  if (slot >= p.out_per) return;
+  const int col = (kvh * p.out_per + slot) * p.out_dv + c;
+  __nv_bfloat16* dst = p.out + static_cast<size_t>(t) * p.out_ld + col;
+  const __nv_bfloat16* gate = p.gate != nullptr ? p.gate + static_cast<size_t>(t) * p.gate_ld + col : nullptr;
+  if (N % 8 == 0 && p.out_vec) {
+#pragma unroll
+    for (int u = 0; u < N / 8; ++u) {
+      if (c + u * 8 < p.out_dv) {  // out_dv is a multiple of 8
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = o[u * 8 + e];
+        if (gate != nullptr) {
+          const uint4 raw = *reinterpret_cast<const uint4*>(gate + u * 8);
+          const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            v[2 * e] *= sigmoid_fast(__uint_as_float(w[e] << 16));
+            v[2 * e + 1] *= sigmoid_fast(__uint_as_float(w[e] & 0xffff0000u));
+          }
+        }
+        *reinterpret_cast<uint4*>(dst + u * 8) = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+      }
+    }
+  } else {
+#pragma unroll
+    for (int e = 0; e < N; ++e)
+      if (c + e < p.out_dv) dst[e] = __float2bfloat16_rn(gate != nullptr ? o[e] * sigmoid_fast(__bfloat162float(gate[e])) : o[e]);
+  }
+}
 // events: 0 K landed (MMA thread)  1 P ready seen by the MMA thread  2 S ready seen by softmax  3 P published  4 partial O read
 #define DSB_PF_TRACE(ev, j) \
   if (tracing && (j) < 64) p.trace[8 + (j) * 8 + (ev)] = clock64();
@@ -309,7 +349,9 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const float slope_l2 = (has_alibi && live) ? p.alibi[kvh * p.group + g] * 1.4426950408889634f : 0.f;
       const bool has_cap = p.cap_l2 > 0.f;  // capped scores are formed in the exp2 domain too
       const bool has_dist = p.r1 != nullptr;  // so is the distance term
-      const float r1h = (has_dist && live) ? p.r1[kvh * p.group + g] : 0.f, r2h = (has_dist && live) ? p.r2[kvh * p.group + g] : 0.f;
+      const bool has_log = p.r2 != nullptr;
+      const float r1h = (has_dist && live) ? p.r1[kvh * p.group + g] * (has_log ? 1.f : 1.4426950408889634f) : 0.f;
+      const float r2h = (has_log && live) ? p.r2[kvh * p.group + g] : 0.f;
       const float sl2 = (has_alibi || has_cap || has_dist) ? 1.f : p.scale_log2;
       __nv_bfloat16* xmax = reinterpret_cast<__nv_bfloat16*>(smem + SMEM::X_OFF);  // [part][row]
       const uint32_t bar_a = 1 + q4, bar_b = 5 + q4;  // the 4 warps (128 threads) that share the rows of this quarter
@@ -365,7 +407,11 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
           for (int i = 0; i < 32; ++i) sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), p.scale_log2, slope_l2 * (key0f + i)));
         }
-        if (has_dist) {  // behind the mask: a hidden key stays at -inf; its (negative) distance is clamped so that the logarithm stays finite
+        if (has_dist && !has_log) {  // r1h (i - j) with the exp2 domain's factor already in r1h
+          const float base = -r1h * static_cast<float>(pos0 + ti - key0);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), p.scale_log2, fmaf(r1h, static_cast<float>(i), base)));
+        } else if (has_dist) {  // behind the mask: a hidden key stays at -inf; its (negative) distance is clamped so that the logarithm stays finite
           const float d0 = static_cast<float>(pos0 + ti - key0);
 #pragma unroll
           for (int i = 0; i < 32; ++i)
@@ -448,6 +494,11 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           if (p.sink > 0.f) l_run += p.sink * exp2f(m_run == -INFINITY ? 0.f : -m_run);  // the sink's score is 0 (splits: added by the merge)
           if (p.sink_logit != nullptr) l_run += exp2f(p.sink_logit[head] * 1.4426950408889634f - (m_run == -INFINITY ? 0.f : m_run));
           const float inv_l = p.out_scale / l_run;
+          if (p.out_dv > 0) {
+#pragma unroll
+            for (int i = 0; i < DQ; ++i) o_acc[i] *= inv_l;
+            store_compact<DQ>(p, t, kvh, g, part * DQ, o_acc);
+          } else {
           __nv_bfloat16* dst = p.out + static_cast<size_t>(t) * p.out_ld + head * D + part * DQ;
 #pragma unroll
           for (int u = 0; u < DQ / 8; ++u) {
@@ -458,6 +509,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             val.z = pack_bf16x2(o[4] * inv_l, o[5] * inv_l);
             val.w = pack_bf16x2(o[6] * inv_l, o[7] * inv_l);
             *reinterpret_cast<uint4*>(dst + u * 8) = val;
+          }
           }
         } else {
           const size_t slot = (static_cast<size_t>(t) * p.hq + head) * p.n_splits + split;
@@ -713,7 +765,7 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       float r1h[CPT], r2h[CPT];       // distance term of the column's head (0 without one)
       const bool has_alibi = p.alibi != nullptr;
       const bool has_cap = p.cap_l2 > 0.f;
-      const bool has_dist = p.r1 != nullptr;
+      const bool has_dist = p.r1 != nullptr, has_log = p.r2 != nullptr;
       const float sl2 = (has_alibi || has_cap || has_dist) ? 1.f : p.scale_log2;
 #pragma unroll
       for (int i = 0; i < CPT; ++i) {
@@ -722,8 +774,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         limit[i] = c0 + i < nq ? pos0 + (c0 + i) / p.group + 1 : 0x3fffffff;
         first[i] = c0 + i >= nq ? 0 : (p.window > 0 ? max(0, limit[i] - p.window) : (p.part > 0 ? ((limit[i] - 1) / p.part) * p.part : 0));
         slope_l2[i] = (has_alibi && c0 + i < nq) ? p.alibi[kvh * p.group + (c0 + i) % p.group] * 1.4426950408889634f : 0.f;
-        r1h[i] = (has_dist && c0 + i < nq) ? p.r1[kvh * p.group + (c0 + i) % p.group] : 0.f;
-        r2h[i] = (has_dist && c0 + i < nq) ? p.r2[kvh * p.group + (c0 + i) % p.group] : 0.f;
+        r1h[i] = (has_dist && c0 + i < nq) ? p.r1[kvh * p.group + (c0 + i) % p.group] * (has_log ? 1.f : 1.4426950408889634f) : 0.f;
+        r2h[i] = (has_log && c0 + i < nq) ? p.r2[kvh * p.group + (c0 + i) % p.group] : 0.f;
       }
       const uint32_t s_addr0 = tmem_base + c0 + lane_off, o_addr = tmem_base + 32 + c0 + lane_off;
       for (int j = 0; j < n_blocks; ++j) {
@@ -743,7 +795,8 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           const float raw = has_cap ? soft_cap_l2(__uint_as_float(sv[i]), p.cap_in, p.cap_l2) : __uint_as_float(sv[i]);
           s[i] = (key >= limit[i] || (key < first[i] && key >= p.keep)) ? -INFINITY : raw;
           if (has_alibi) s[i] = fmaf(s[i], p.scale_log2, slope_l2[i] * static_cast<float>(key));
-          if (has_dist) s[i] = fmaf(s[i], p.scale_log2, -r1h[i] * __log2f(fmaf(r2h[i], fmaxf(static_cast<float>(limit[i] - 1 - key), 0.f), 1.f)));
+          if (has_dist && !has_log) s[i] = fmaf(s[i], p.scale_log2, -r1h[i] * static_cast<float>(limit[i] - 1 - key));
+          else if (has_dist) s[i] = fmaf(s[i], p.scale_log2, -r1h[i] * __log2f(fmaf(r2h[i], fmaxf(static_cast<float>(limit[i] - 1 - key), 0.f), 1.f)));
           const uint32_t bits = __float_as_uint(s[i]);
           const uint32_t r = __reduce_max_sync(0xffffffffu, bits ^ ((bits >> 31) ? 0xffffffffu : 0x80000000u));
           wm[i] = __uint_as_float(r ^ ((r >> 31) ? 0x80000000u : 0xffffffffu));
@@ -827,7 +880,9 @@ paged_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           if (!partial) {
             if (p.sink > 0.f) l += p.sink * exp2f(m_run[i] == -INFINITY ? 0.f : -m_run[i]);  // the sink's score is 0 (splits: added by the merge)
             if (p.sink_logit != nullptr) l += exp2f(p.sink_logit[head] * 1.4426950408889634f - (m_run[i] == -INFINITY ? 0.f : m_run[i]));
-            p.out[static_cast<size_t>(t) * p.out_ld + head * D + row] = __float2bfloat16_rn(__uint_as_float(ov[i]) / l * p.out_scale);
+            const float o = __uint_as_float(ov[i]) / l * p.out_scale;
+            if (p.out_dv > 0) store_compact<1>(p, t, kvh, c % p.group, row, &o);
+            else p.out[static_cast<size_t>(t) * p.out_ld + head * D + row] = __float2bfloat16_rn(o);
           } else {
             const size_t slot = (static_cast<size_t>(t) * p.hq + head) * p.n_splits + split;
             p.part_o[slot * D + row] = __uint_as_float(ov[i]);
@@ -862,13 +917,17 @@ struct MaskExtras {
   const float* r1 = nullptr;
   const float* r2 = nullptr;
   int part = 0;
+  int out_dv = 0, out_per = 0;
+  const __nv_bfloat16* gate = nullptr;
+  long long gate_ld = 0;
 };
 
 // out[t][h][:] = sum_s 2^(m_s - M) O_s / sum_s 2^(m_s - M) l_s ; one warp per (token, head)
 template <int D>
-__global__ void combine_splits_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
-                                      int rows, int n_splits, int hq, long long out_ld, float out_scale, float sink,
-                                      const float* __restrict__ sink_logit) {
+__global__ void combine_splits_kernel(const Params p, int rows) {
+  const float *part_o = p.part_o, *part_ml = p.part_ml, *sink_logit = p.sink_logit;
+  const int n_splits = p.n_splits, hq = p.hq;
+  const float sink = p.sink;
   const int wid = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (wid >= rows) return;
   constexpr int EPL = D / 32;
@@ -889,8 +948,14 @@ __global__ void combine_splits_kernel(const float* __restrict__ part_o, const fl
   }
   if (sink > 0.f) L += sink * exp2f(M == -INFINITY ? 0.f : -M);  // a softmax with a sink: its score is 0
   if (sink_logit != nullptr) L += exp2f(sink_logit[wid % hq] * 1.4426950408889634f - (M == -INFINITY ? 0.f : M));  // a learned sink per head
-  const float inv = out_scale / L;
-  __nv_bfloat16* dst = out + static_cast<size_t>(wid / hq) * out_ld + (wid % hq) * D;
+  const float inv = p.out_scale / L;
+  if (p.out_dv > 0) {
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) acc[e] *= inv;
+    store_compact<EPL>(p, wid / hq, (wid % hq) / p.group, (wid % hq) % p.group, lane * EPL, acc);
+    return;
+  }
+  __nv_bfloat16* dst = p.out + static_cast<size_t>(wid / hq) * p.out_ld + (wid % hq) * D;
 #pragma unroll
   for (int e = 0; e < EPL; ++e) dst[lane * EPL + e] = __float2bfloat16_rn(acc[e] * inv);
 }
@@ -946,6 +1011,8 @@ static int launch(const void* qkv, const void* kv_cache, void* out, const int* t
   p.keep = window > 0 ? keep : 0; p.out_ld = out_ld ? out_ld : static_cast<long long>(hq) * D; p.out_scale = out_scale;
   p.cap_l2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   p.sink = sink; p.sink_logit = ex.sink_logit; p.r1 = ex.r1; p.r2 = ex.r2; p.part = window > 0 ? 0 : ex.part;
+  p.out_dv = ex.out_dv; p.out_per = ex.out_per; p.gate = ex.gate; p.gate_ld = ex.gate_ld;
+  p.out_vec = ex.out_dv % 8 == 0 && p.out_ld % 8 == 0 && ex.gate_ld % 8 == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(ex.gate)) & 15) == 0;
   static const bool want_trace = [] { const char* e = getenv("DSB200_PF_TRACE"); return e && atoi(e) != 0; }();
   static long long* trace_buf = nullptr;
   p.trace = nullptr;
@@ -969,8 +1036,7 @@ static int launch(const void* qkv, const void* kv_cache, void* out, const int* t
   }
   if (n_splits > 1) {
     const int rows = T * hq;
-    combine_splits_kernel<D><<<(rows * 32 + 255) / 256, 256, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), rows, n_splits, hq, p.out_ld,
-                                                                          p.out_scale, p.sink, p.sink_logit);
+    combine_splits_kernel<D><<<(rows * 32 + 255) / 256, 256, 0, stream>>>(p, rows);
     DSB_CHECK_CUDA(cudaGetLastError());
   }
   return DSB_OK;
@@ -1020,6 +1086,8 @@ static int launch_decode(const void* qkv, const void* kv_cache, void* out, const
   p.keep = window > 0 ? keep : 0; p.out_ld = out_ld ? out_ld : static_cast<long long>(hq) * D; p.out_scale = out_scale;
   p.cap_l2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   p.sink = sink; p.sink_logit = ex.sink_logit; p.r1 = ex.r1; p.r2 = ex.r2; p.part = window > 0 ? 0 : ex.part;
+  p.out_dv = ex.out_dv; p.out_per = ex.out_per; p.gate = ex.gate; p.gate_ld = ex.gate_ld;
+  p.out_vec = ex.out_dv % 8 == 0 && p.out_ld % 8 == 0 && ex.gate_ld % 8 == 0 && ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(ex.gate)) & 15) == 0;
   static const bool want_trace = [] { const char* e = getenv("DSB200_PF_TRACE"); return e && atoi(e) != 0; }();
   static long long* trace_buf = nullptr;
   if (want_trace) {
@@ -1042,8 +1110,7 @@ static int launch_decode(const void* qkv, const void* kv_cache, void* out, const
   }
   if (n_splits > 1) {
     const int rows = T * hq;
-    combine_splits_kernel<D><<<(rows * 32 + 255) / 256, 256, 0, stream>>>(part_o, part_ml, static_cast<__nv_bfloat16*>(out), rows, n_splits, hq, p.out_ld,
-                                                                          p.out_scale, p.sink, p.sink_logit);
+    combine_splits_kernel<D><<<(rows * 32 + 255) / 256, 256, 0, stream>>>(p, rows);
     DSB_CHECK_CUDA(cudaGetLastError());
   }
   return DSB_OK;
@@ -1106,14 +1173,17 @@ DSB_EXPORT int dsb200_paged_flash_decode(const void* qkv, const void* kv_cache, 
 // out is [n_tokens][heads][rank] bf16; rank 64 or 128.  decode != 0 selects the small-atom kernel (rank 128, heads dividing 16).
 // Scratch and atoms as for dsb200_paged_flash_attention with hq = heads.
 // sink_logit (null, or `heads` floats): exp(sink_logit[h]) joins head h's softmax denominator, an entry without key and value.
+// window > 0: a query at position i sees only the rows with i - j < window (only their pages are visited); 0 = the whole history.
 DSB_EXPORT int dsb200_paged_flash_latent_sink(const void* q, int q_heads, long long q_head_stride, long long q_tok_stride, const void* cache,
                                               void* out, const int* tok_seq, const int* tok_pos, const int* block_table, int n_tokens, int heads,
                                               int rank, int block_size, int max_blocks_per_seq, int num_blocks, float scale,
-                                              const float* sink_logit, int max_atoms, int n_splits, void* scratch, int decode, cudaStream_t stream) {
+                                              const float* sink_logit, int window, int max_atoms, int n_splits, void* scratch, int decode,
+                                              cudaStream_t stream) {
   using namespace dsb;
   if (n_tokens == 0) return DSB_OK;
   paged::MaskExtras ex;
   ex.sink_logit = sink_logit;
+  DSB_REQUIRE(window >= 0, "paged_flash_latent: window %d", window);
   DSB_REQUIRE(rank == 64 || rank == 128, "paged_flash_latent: rank %d unsupported (64 or 128)", rank);
   DSB_REQUIRE(heads >= 1 && 128 % heads == 0 && q_heads >= 1 && q_heads <= heads, "paged_flash_latent: %d (%d given) heads must divide 128", heads, q_heads);
   DSB_REQUIRE(q_head_stride % 8 == 0 && q_tok_stride % 8 == 0 && q_head_stride > 0 && q_tok_stride > 0, "paged_flash_latent: query strides must be multiples of 8 elements");
@@ -1122,13 +1192,13 @@ DSB_EXPORT int dsb200_paged_flash_latent_sink(const void* q, int q_heads, long l
   if (decode) {
     DSB_REQUIRE(rank == 128 && 16 % heads == 0, "paged_flash_latent: the small-atom kernel takes rank 128 and heads dividing 16");
     return paged::launch_decode(q, cache, out, tok_seq, tok_pos, block_table, n_tokens, heads, 1, block_size, max_blocks_per_seq, num_blocks,
-                                scale, max_atoms, n_splits, scratch, nullptr, 0, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
+                                scale, max_atoms, n_splits, scratch, nullptr, window, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
   }
   if (rank == 128)
     return paged::launch<128>(q, cache, out, tok_seq, tok_pos, block_table, n_tokens, heads, 1, block_size, max_blocks_per_seq, num_blocks,
-                              scale, max_atoms, n_splits, scratch, nullptr, 0, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
+                              scale, max_atoms, n_splits, scratch, nullptr, window, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
   return paged::launch<64>(q, cache, out, tok_seq, tok_pos, block_table, n_tokens, heads, 1, block_size, max_blocks_per_seq, num_blocks, scale,
-                           max_atoms, n_splits, scratch, nullptr, 0, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
+                           max_atoms, n_splits, scratch, nullptr, window, stream, q_heads, q_head_stride, q_tok_stride, 1, 0, 0, 1.f, 0.f, 0.f, ex);
 }
 
 DSB_EXPORT int dsb200_paged_flash_latent(const void* q, int q_heads, long long q_head_stride, long long q_tok_stride, const void* cache,
@@ -1136,7 +1206,7 @@ DSB_EXPORT int dsb200_paged_flash_latent(const void* q, int q_heads, long long q
                                          int rank, int block_size, int max_blocks_per_seq, int num_blocks, float scale, int max_atoms,
                                          int n_splits, void* scratch, int decode, cudaStream_t stream) {
   return dsb200_paged_flash_latent_sink(q, q_heads, q_head_stride, q_tok_stride, cache, out, tok_seq, tok_pos, block_table, n_tokens, heads, rank,
-                                        block_size, max_blocks_per_seq, num_blocks, scale, nullptr, max_atoms, n_splits, scratch, decode, stream);
+                                        block_size, max_blocks_per_seq, num_blocks, scale, nullptr, 0, max_atoms, n_splits, scratch, decode, stream);
 }
 
 // Sliding-window attention that keeps the first keys visible, on the tensor-core kernels: a query at position p sees the keys j <= p with
@@ -1173,23 +1243,30 @@ DSB_EXPORT int dsb200_paged_flash_window(const void* q, long long q_tok_stride, 
 // bf16 at q_tok_stride elements per token (a multiple of 8), kv_cache [num_blocks][2][block_size][hkv][head_dim] bf16; out rows at out_ld
 // elements per token (a multiple of 8).  decode != 0 selects the small-atom kernel (head_dim 128, q:kv head ratios dividing 16).
 // sink_logit (hq floats): learned sinks, exp(sink_logit[h]) joins head h's denominator; r1, r2 (hq floats each): the score of key j for the
-// query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions;
-// window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0).
+// query at position i loses r1[h] ln(1 + r2[h] (i - j)), r1 alone: it loses r1[h] (i - j); part > 0: a query sees only the keys of its own part of
+// `part` positions; window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0).
+// out_dv > 0: compact output -- of every group of hq / hkv slots only the first out_per are heads, and only the first out_dv entries of a head leave:
+// out row [hkv * out_per][out_dv]; gate (null, or bf16 [n_tokens][gate_ld] in that layout): the output times the sigmoid of it.
 DSB_EXPORT int dsb200_paged_flash_sink_ex(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld, const int* tok_seq,
                                        const int* tok_pos, const int* block_table, int n_tokens, int hq, int hkv, int head_dim, int block_size,
                                        int max_blocks_per_seq, int num_blocks, float scale, float softcap, float sink, const float* sink_logit,
-                                       const float* r1, const float* r2, int part, int window, int max_atoms, int n_splits, void* scratch, int decode,
-                                       cudaStream_t stream) {
+                                       const float* r1, const float* r2, int part, int window, int out_dv, int out_per, const void* gate, long long gate_ld,
+                                       int max_atoms, int n_splits, void* scratch, int decode, cudaStream_t stream) {
   using namespace dsb;
   if (n_tokens == 0) return DSB_OK;
-  DSB_REQUIRE((r1 == nullptr) == (r2 == nullptr) && part >= 0 && window >= 0 && (part == 0 || window == 0) && (r1 == nullptr || softcap == 0.f),
+  DSB_REQUIRE((r1 != nullptr || r2 == nullptr) && part >= 0 && window >= 0 && (part == 0 || window == 0) && (r1 == nullptr || softcap == 0.f),
               "paged_flash_sink: distance term / part %d / window %d", part, window);
   paged::MaskExtras ex;
   ex.sink_logit = sink_logit; ex.r1 = r1; ex.r2 = r2; ex.part = part;
+  ex.out_dv = out_dv; ex.out_per = out_per; ex.gate = static_cast<const __nv_bfloat16*>(gate); ex.gate_ld = gate_ld;
+  DSB_REQUIRE(out_dv >= 0 && out_dv <= head_dim && (out_dv > 0 || gate == nullptr) && (out_dv == 0 || (out_per >= 1 && out_per <= hq / hkv)) &&
+                  (gate == nullptr || gate_ld >= static_cast<long long>(hkv) * out_per * out_dv),
+              "paged_flash_sink: compact output of %d x %d, gate stride %lld", out_per, out_dv, gate_ld);
   DSB_REQUIRE(head_dim == 64 || head_dim == 128, "paged_flash_sink: head_dim %d unsupported (64 or 128)", head_dim);
   DSB_REQUIRE(hq % hkv == 0 && 128 % (hq / hkv) == 0, "paged_flash_sink: q/kv head ratio %d must divide 128", hq / hkv);
   DSB_REQUIRE(block_size >= 8 && block_size <= 128 && 128 % block_size == 0, "paged_flash_sink: KV block size %d must divide 128", block_size);
-  DSB_REQUIRE(softcap >= 0.f && sink >= 0.f && q_tok_stride % 8 == 0 && out_ld % 8 == 0 && out_ld >= static_cast<long long>(hq) * head_dim,
+  DSB_REQUIRE(softcap >= 0.f && sink >= 0.f && q_tok_stride % 8 == 0 &&
+                  (out_dv > 0 ? out_ld >= static_cast<long long>(hkv) * out_per * out_dv : (out_ld % 8 == 0 && out_ld >= static_cast<long long>(hq) * head_dim)),
               "paged_flash_sink: cap %f, sink %f, strides %lld / %lld", softcap, sink, q_tok_stride, out_ld);
   DSB_REQUIRE(max_atoms >= 1 && n_splits >= 1 && n_splits <= 64 && scratch != nullptr, "paged_flash_sink: bad max_atoms / n_splits / scratch");
   if (decode) {
@@ -1209,6 +1286,6 @@ DSB_EXPORT int dsb200_paged_flash_sink(const void* q, long long q_tok_stride, co
                                        int max_blocks_per_seq, int num_blocks, float scale, float softcap, float sink, int max_atoms, int n_splits,
                                        void* scratch, int decode, cudaStream_t stream) {
   return dsb200_paged_flash_sink_ex(q, q_tok_stride, kv_cache, out, out_ld, tok_seq, tok_pos, block_table, n_tokens, hq, hkv, head_dim, block_size,
-                                    max_blocks_per_seq, num_blocks, scale, softcap, sink, nullptr, nullptr, nullptr, 0, 0, max_atoms, n_splits, scratch,
+                                    max_blocks_per_seq, num_blocks, scale, softcap, sink, nullptr, nullptr, nullptr, 0, 0, 0, 0, nullptr, 0, max_atoms, n_splits, scratch,
                                     decode, stream);
 }

@@ -16,6 +16,7 @@
 //   grouped_topk_gating   softmax scores (+ correction for the selection only), best `keep` of `groups` contiguous expert groups by
 //                         their largest selection score, top-k of the surviving experts, weights = uncorrected scores
 //   moe_scatter / moe_gather   expert-sorted copies and the weighted fp32 combine, any width
+//   gelu_gate_cols        gelu(g) * u (tanh form)
 //   clamped_swish_gate    min(g, L) * sigmoid(alpha * min(g, L)) * (clamp(u, -L, L) + shift)
 //   moe_gemm_rows         grouped expert GEMM on CUDA cores (fp32 accumulation) for shapes / dtypes the tensor-core
 //                         grouped GEMM does not take
@@ -649,6 +650,43 @@ __global__ void clamped_swish_gate_cols_vec_kernel(const T* __restrict__ gu, lon
   }
 }
 
+// The gate of gelu-gated feed-forwards on column ranges, like clamped_swish_gate_cols: out = gelu(g) * u with the tanh form of gelu,
+// 0.5 z (1 + tanh(w)) = z / (1 + exp(-2 w)), w = sqrt(2 / pi) (z + 0.044715 z^3): one exponential and one division per value.  A bf16 result takes
+// the fast ones (their error is far below its rounding).
+template <typename T>
+__device__ __forceinline__ float gelu_gate_one(float z, float u);
+template <>
+__device__ __forceinline__ float gelu_gate_one<float>(float z, float u) {
+  return z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))) * u;
+}
+template <>
+__device__ __forceinline__ float gelu_gate_one<bf16>(float z, float u) {
+  const float e = __expf(fminf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z), 80.f));  // __fdividef wants a denominator below 2^126
+  return __fdividef(z, 1.f + e) * u;
+}
+template <typename T>
+__global__ void gelu_gate_cols_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, T* __restrict__ out, long long out_ld, long long rows,
+                                      int F) {
+  const long long n = rows * F;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / F;
+    const int c = static_cast<int>(i % F);
+    out[r * out_ld + c] = from_f<T>(gelu_gate_one<T>(to_f(gu[r * ld + gate_col0 + c]), to_f(gu[r * ld + up_col0 + c])));
+  }
+}
+template <typename T>
+__global__ void gelu_gate_cols_vec_kernel(const T* __restrict__ gu, long long ld, int gate_col0, int up_col0, T* __restrict__ out, long long out_ld,
+                                          long long rows, int F) {
+  const int fv = F >> 2;
+  const long long n = rows * fv;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const long long r = i / fv;
+    const int c = static_cast<int>(i % fv) * 4;
+    const float4 g = load4(gu + r * ld + gate_col0 + c), u = load4(gu + r * ld + up_col0 + c);
+    store4(out + r * out_ld + c, make_float4(gelu_gate_one<T>(g.x, u.x), gelu_gate_one<T>(g.y, u.y), gelu_gate_one<T>(g.z, u.z), gelu_gate_one<T>(g.w, u.w)));
+  }
+}
+
 __global__ void softcap_kernel(float* __restrict__ x, long long ld, int cols, long long n, float cap) {
   for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x) {
     float* p = x + (i / cols) * ld + (i % cols);
@@ -1131,6 +1169,26 @@ DSB_EXPORT int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int 
   else
     clamped_swish_gate_cols_kernel<float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, row_col, (float*)out, out_ld, rows, F,
                                                                                alpha, limit, shift);
+  DSB_CHECK_CUDA(cudaGetLastError());
+  return DSB_OK;
+}
+
+// out[r, c] = gelu(gu[r, gate_col0 + c]) * gu[r, up_col0 + c] (tanh form of gelu) for c < F; gu [rows, ld], out [rows, out_ld]; dtype 0 = bf16, 1 = fp32.
+DSB_EXPORT int dsb200_gelu_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, void* out, long long out_ld, long long rows, int F,
+                                     int dtype, cudaStream_t stream) {
+  const long long n = rows * F;
+  if (n == 0) return DSB_OK;
+  const int esz = dtype == 0 ? 2 : 4;
+  const bool vec = F % 4 == 0 && gate_col0 % 4 == 0 && up_col0 % 4 == 0 && ld % 4 == 0 && out_ld % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & (4 * esz - 1)) == 0;
+  if (vec && dtype == 0)
+    gelu_gate_cols_vec_kernel<bf16><<<grid_for(n / 4, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, (bf16*)out, out_ld, rows, F);
+  else if (vec)
+    gelu_gate_cols_vec_kernel<float><<<grid_for(n / 4, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, (float*)out, out_ld, rows, F);
+  else if (dtype == 0)
+    gelu_gate_cols_kernel<bf16><<<grid_for(n, 256), 256, 0, stream>>>((const bf16*)gu, ld, gate_col0, up_col0, (bf16*)out, out_ld, rows, F);
+  else
+    gelu_gate_cols_kernel<float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)gu, ld, gate_col0, up_col0, (float*)out, out_ld, rows, F);
   DSB_CHECK_CUDA(cudaGetLastError());
   return DSB_OK;
 }

@@ -161,13 +161,16 @@ __global__ void head_norm_rotary_append_kernel(const T* __restrict__ proj, long 
 // sequence, and strides of their own for query / output heads and cached rows (so that one cached row can serve as key and as value).
 struct SinkExtras {
   const float* sink_logit;     // [H] or null: exp(sink_logit[h]) joins the denominator (an entry without key and value)
-  const float* r1;             // [H] or null: the score of key j loses r1[h] ln(1 + r2[h] (pos - j))
+  const float* r1;             // [H] or null: the score of key j loses r1[h] ln(1 + r2[h] (pos - j)), or r1[h] (pos - j) when r2 is null
   const float* r2;
   int part;                    // > 0: a query at pos sees only the keys j <= pos with j / part == pos / part
   int window;                  // > 0: a query at pos sees only the keys j <= pos with pos - j < window
   int k_row, v_row;            // elements between the heads of a cached key row / value row (>= d, dv)
   long long q_head_stride;     // elements between the heads of a query row
   long long out_head_stride;   // elements between the heads of an output row
+  int q_group;                 // slots per key / value head in a query row (>= H / G): head h lies in slot (h / (H / G)) q_group + h % (H / G)
+  const void* gate;            // null, or gate pre-activations in the activation dtype: entry c of head h is multiplied by
+  long long gate_ld;           //   sigmoid(gate[t * gate_ld + h * dv + c]) before it is rounded
 };
 
 // One block per (token, query head).  The visible keys first .. pos are walked in chunks of SA_CHUNK with a running maximum / sum (fp32).
@@ -182,17 +185,17 @@ sink_attention_kernel(const T* __restrict__ q, long long q_ld, const T* __restri
   __shared__ float red[33];
   __shared__ float sc[SA_CHUNK];
   __shared__ int key_blk[SA_CHUNK], key_slot[SA_CHUNK];
-  const int t = blockIdx.x, h = blockIdx.y, g = h / (H / G);
+  const int t = blockIdx.x, h = blockIdx.y, per = H / G, g = h / per, q_slot = g * ex.q_group + h % per;
   const int seq = tok_seq[t], pos = tok_pos[t];
   float* qs = sm;        // [d]
   float* acc = sm + d;   // [dv]
-  for (int c = threadIdx.x; c < d; c += SA_THREADS) qs[c] = to_f(q[static_cast<long long>(t) * q_ld + h * ex.q_head_stride + c]) * scale;
+  for (int c = threadIdx.x; c < d; c += SA_THREADS) qs[c] = to_f(q[static_cast<long long>(t) * q_ld + q_slot * ex.q_head_stride + c]) * scale;
   for (int c = threadIdx.x; c < dv; c += SA_THREADS) acc[c] = 0.f;
   const int n = pos + 1;
   const int first = max(ex.part > 0 ? (pos / ex.part) * ex.part : 0, ex.window > 0 ? pos + 1 - ex.window : 0);
   const int* bt = block_table + static_cast<size_t>(seq) * bt_stride;
   const float inv_cap = cap > 0.f ? 1.f / cap : 0.f;
-  const float r1 = ex.r1 ? ex.r1[h] : 0.f, r2 = ex.r1 ? ex.r2[h] : 0.f;
+  const float r1 = ex.r1 ? ex.r1[h] : 0.f, r2 = ex.r2 ? ex.r2[h] : 0.f;
   // a learned sink starts the running softmax as an entry of its own: maximum = its score, sum = 1, nothing accumulated
   float m_run = ex.sink_logit ? ex.sink_logit[h] : -INFINITY, l_run = ex.sink_logit ? 1.f : 0.f;
   __syncthreads();
@@ -208,7 +211,8 @@ sink_attention_kernel(const T* __restrict__ q, long long q_ld, const T* __restri
       float s = 0.f;
       for (int c = 0; c < d; ++c) s = fmaf(qs[c], to_f(kr[c]), s);
       if (cap > 0.f) s = cap * tanhf(s * inv_cap);
-      if (ex.r1) s -= r1 * log1pf(r2 * static_cast<float>(pos - j));
+      if (ex.r2) s -= r1 * log1pf(r2 * static_cast<float>(pos - j));
+      else if (ex.r1) s -= r1 * static_cast<float>(pos - j);
       sc[x] = s;
       mx = fmaxf(mx, s);
     }
@@ -233,23 +237,28 @@ sink_attention_kernel(const T* __restrict__ q, long long q_ld, const T* __restri
     __syncthreads();
   }
   const float inv = 1.f / (l_run + sink * expf(-m_run));  // the constant sink's score is 0: exp(0 - m) in the shifted sum
-  for (int c = threadIdx.x; c < dv; c += SA_THREADS) out[static_cast<long long>(t) * out_ld + h * ex.out_head_stride + c] = from_f<T>(acc[c] * inv);
+  const T* gate = ex.gate ? static_cast<const T*>(ex.gate) + static_cast<long long>(t) * ex.gate_ld + h * dv : nullptr;
+  for (int c = threadIdx.x; c < dv; c += SA_THREADS) {
+    const float o = acc[c] * inv;
+    out[static_cast<long long>(t) * out_ld + h * ex.out_head_stride + c] = from_f<T>(gate ? o / (1.f + expf(-to_f(gate[c]))) : o);
+  }
 }
 
 // One warp per (token, slot).  Slots 0 .. H - 1: the rotated part (the last dr entries) of query head h, rotated in place.  Slot H: the
 // low-rank row -- its first R entries RMS-normed with a weight, its last dr entries rotated -- goes to the token's row of the cache.
+// Pairs are (i, i + rot / 2), or neighbours (2i, 2i + 1) when `interleaved`.
 template <typename T>
-__device__ __forceinline__ void rotate_half_row(const T* __restrict__ src, T* __restrict__ dst, int n, int rot, int pos, const double* __restrict__ freq,
-                                                int lane) {
+__device__ __forceinline__ void rotate_row(const T* src, T* dst, int n, int rot, int pos, const double* __restrict__ freq, int lane, int interleaved) {
   const int half = rot >> 1;
   for (int i = lane; i < half; i += 32) {
-    const float u = to_f(src[i]), v = to_f(src[i + half]);
+    const int iu = interleaved ? 2 * i : i, iv = interleaved ? 2 * i + 1 : i + half;
+    const float u = to_f(src[iu]), v = to_f(src[iv]);
     double a = static_cast<double>(pos) * freq[i];
     a -= 6.283185307179586476925 * rint(a * 0.15915494309189533576888);  // into [-pi, pi] before single precision takes over
     float sn, cs;
     sincosf(static_cast<float>(a), &sn, &cs);
-    dst[i] = from_f<T>(u * cs - v * sn);
-    dst[i + half] = from_f<T>(v * cs + u * sn);
+    dst[iu] = from_f<T>(u * cs - v * sn);
+    dst[iv] = from_f<T>(v * cs + u * sn);
   }
   if (dst != src)
     for (int c = rot + lane; c < n; c += 32) dst[c] = src[c];
@@ -258,7 +267,7 @@ template <typename T>
 __global__ void latent_rotary_append_kernel(T* __restrict__ proj, long long ld, int q_col0, int kv_col0, const float* __restrict__ wkv,
                                             const double* __restrict__ freq, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                             const int* __restrict__ block_table, int bt_stride, int block_size, T* __restrict__ cache, int row_w,
-                                            int n_tokens, int H, int d, int dr, int R, int rot, float eps) {
+                                            int n_tokens, int H, int d, int dr, int R, int rot, float eps, int interleaved) {
   const int gw = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (gw >= n_tokens * (H + 1)) return;
   const int t = gw / (H + 1), slot = gw % (H + 1);
@@ -266,7 +275,7 @@ __global__ void latent_rotary_append_kernel(T* __restrict__ proj, long long ld, 
   T* row = proj + static_cast<long long>(t) * ld;
   if (slot < H) {
     T* v = row + q_col0 + slot * (d + dr) + d;
-    rotate_half_row(v, v, dr, rot, pos, freq, lane);
+    rotate_row(v, v, dr, rot, pos, freq, lane, interleaved);
     return;
   }
   const T* low = row + kv_col0;
@@ -277,7 +286,7 @@ __global__ void latent_rotary_append_kernel(T* __restrict__ proj, long long ld, 
   s = warp_sum(s);
   const float inv = 1.f / sqrtf(s / static_cast<float>(R) + eps);
   for (int c = lane; c < R; c += 32) dst[c] = from_f<T>(to_f(low[c]) * inv * wkv[c]);
-  rotate_half_row(low + R, dst + R, dr, rot, pos, freq, lane);
+  rotate_row(low + R, dst + R, dr, rot, pos, freq, lane, interleaved);
   for (int c = R + dr + lane; c < row_w; c += 32) dst[c] = from_f<T>(0.f);  // rows padded to a width the tensor-core kernels take
 }
 
@@ -298,7 +307,8 @@ __device__ __forceinline__ void store4(bf16* p, float4 v) {
   *reinterpret_cast<bf16x4*>(p) = o;
 }
 
-// One warp per (token, SL consecutive head slots): the H query heads, then the G key heads, then the G value heads of the token.  Every
+// One warp per (token, SL consecutive head slots): the G q_group query slots, then the G key heads, then the G value heads of the token (has_kv =
+// 0: the layer reads another layer's cache, only its queries are prepared).  Every
 // channel first passes a short causal convolution over the sequence (bias added to every real row; rows before this step's come from the
 // state, rows before the sequence are zeros); query / key heads then get their RMS norm, value heads are mixed with another layer's values of
 // the same token.  A lane owns VEC neighbouring channels at a time (VEC = 4: every size, offset and stride is a multiple of 4 and the rows
@@ -315,17 +325,18 @@ conv_head_norm_append_kernel(const T* __restrict__ proj, long long ld, int col0,
                              const int* __restrict__ block_table, int bt_stride, int block_size, T* __restrict__ k_cache, long long k_block_stride,
                              T* __restrict__ v_cache, long long v_block_stride, T* __restrict__ q_out, long long q_ld, const T* __restrict__ v_other,
                              const float* __restrict__ mix, T* __restrict__ v_own, int n_tokens, int H, int G, int d, int dv, int taps, float eps,
-                             int q_row, int k_row, int v_row) {
+                             int q_row, int k_row, int v_row, int q_group, int has_kv) {
   const int gw = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-  const int per_tok = H + 2 * G, groups = (per_tok + SL - 1) / SL;
+  const int n_q = G * q_group, per = H / G;
+  const int per_tok = n_q + (has_kv ? 2 * G : 0), groups = (per_tok + SL - 1) / SL;
   if (gw >= n_tokens * groups) return;
   const int t = gw / groups, slot0 = (gw % groups) * SL;
   const int seq = tok_seq[t], pos = tok_pos[t];
   const int4 sd = seq_desc[seq];
   const int i = t - sd.x;  // index among the sequence's new tokens
-  const int C = (H + G) * d + G * dv;  // convolved channels: q | k | v, as they lie in proj from col0 on and in the state rows
+  const int C = H * d + (has_kv ? G * (d + dv) : 0);  // convolved channels: q | k | v (or q), as they lie in proj from col0 on and in the state rows
   const T* st = state ? state + static_cast<size_t>(sd.w) * (taps - 1) * C : nullptr;
-  const long long cache_row = block_table[static_cast<size_t>(seq) * bt_stride + pos / block_size];
+  const long long cache_row = has_kv ? block_table[static_cast<size_t>(seq) * bt_stride + pos / block_size] : 0;
   const int in_block = pos % block_size;
   // rows the taps read: tap j reads the token taps - 1 - j positions back -- a row of this step, a row of the state, or nothing
   const int j0 = max(0, taps - 1 - pos);           // taps before j0 lie before the sequence's start
@@ -340,13 +351,13 @@ conv_head_norm_append_kernel(const T* __restrict__ proj, long long ld, int col0,
   };
   auto slot_of = [&](int slot) {
     Slot o;
-    o.is_q = slot < H;
-    o.is_v = slot >= H + G;
-    o.head = o.is_q ? slot : (o.is_v ? slot - H - G : slot - H);
-    o.n = o.is_v ? dv : d;
+    o.is_q = slot < n_q;
+    o.is_v = slot >= n_q + G;
+    o.head = o.is_q ? (slot / q_group) * per + slot % q_group : (o.is_v ? slot - n_q - G : slot - n_q);
+    o.n = o.is_v ? dv : (o.is_q && slot % q_group >= per ? 0 : d);  // 0: a slot without a head, all zeros
     o.ch0 = o.is_q ? o.head * d : (o.is_v ? (H + G) * d + o.head * dv : H * d + o.head * d);
     o.width = o.is_q ? q_row : (o.is_v ? v_row : k_row);
-    o.dst = o.is_q ? q_out + static_cast<long long>(t) * q_ld + o.head * q_row
+    o.dst = o.is_q ? q_out + static_cast<long long>(t) * q_ld + slot * q_row
                    : (o.is_v ? v_cache + cache_row * v_block_stride + (static_cast<long long>(in_block) * G + o.head) * v_row
                              : k_cache + cache_row * k_block_stride + (static_cast<long long>(in_block) * G + o.head) * k_row);
     return o;
@@ -395,12 +406,12 @@ conv_head_norm_append_kernel(const T* __restrict__ proj, long long ld, int col0,
         for (int e = 0; e < VEC; ++e) o[e] = y[e];
       }
     } else {
-      const float* w = S.is_q ? wq : wk;
+      const float* w = S.is_q ? wq : wk;  // null: the norm has no weight
       if constexpr (VEC == 4) {
-        const float4 g = load4(w + c);
+        const float4 g = w ? load4(w + c) : make_float4(1.f, 1.f, 1.f, 1.f);
         o[0] = y[0] * inv * g.x; o[1] = y[1] * inv * g.y; o[2] = y[2] * inv * g.z; o[3] = y[3] * inv * g.w;
       } else {
-        o[0] = y[0] * inv * w[c];
+        o[0] = y[0] * inv * (w ? w[c] : 1.f);
       }
     }
     if constexpr (VEC == 4) store4(S.dst + c, make_float4(o[0], o[1], o[2], o[3]));
@@ -429,7 +440,7 @@ conv_head_norm_append_kernel(const T* __restrict__ proj, long long ld, int col0,
         float inv = 1.f;
         if (!S.is_v) {
           ss = warp_sum(ss);
-          inv = 1.f / sqrtf(ss / static_cast<float>(S.n) + eps);
+          inv = 1.f / sqrtf(ss / static_cast<float>(max(S.n, 1)) + eps);
         }
         if (c < S.n) emit(S, c, held[s], inv);
         for (int x = S.n + lane; x < S.width; x += 32) S.dst[x] = from_f<T>(0.f);  // padding: adds nothing to a score or an output
@@ -458,7 +469,7 @@ conv_head_norm_append_kernel(const T* __restrict__ proj, long long ld, int col0,
     float inv = 1.f;
     if (!S.is_v) {
       ss = warp_sum(ss);
-      inv = 1.f / sqrtf(ss / static_cast<float>(S.n) + eps);
+      inv = 1.f / sqrtf(ss / static_cast<float>(max(S.n, 1)) + eps);
     }
 #pragma unroll
     for (int k = 0; k < GROUPS; ++k) {
@@ -546,39 +557,43 @@ DSB_EXPORT int dsb200_sink_attention(const void* q, long long q_ld, const void* 
   if (n_tokens == 0) return DSB_OK;
   DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && d >= 1 && dv >= 1 && d + dv <= 8192 && sink >= 0.f, "sink_attention: heads %d / %d, head sizes %d / %d", H, G,
               d, dv);
-  const SinkExtras ex{nullptr, nullptr, nullptr, 0, 0, d, dv, d, dv};
+  const SinkExtras ex{nullptr, nullptr, nullptr, 0, 0, d, dv, d, dv, H / G, nullptr, 0};
   return launch_sink_attention(q, q_ld, k_cache, k_block_stride, v_cache, v_block_stride, tok_seq, tok_pos, block_table, bt_stride, block_size, out,
                                out_ld, n_tokens, H, G, d, dv, scale, cap, sink, ex, dtype, stream);
 }
 
 // `sink_attention` with learned sinks, a distance term, a mask by parts and free strides:
 //   sink_logit [H] (or null): exp(sink_logit[h]) joins head h's denominator;   r1, r2 [H] (or both null): s_j -= r1[h] ln(1 + r2[h] (pos - j));
+//   r1 alone: s_j -= r1[h] (pos - j);
 //   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible; window > 0: only
 //   the keys with pos - j < window;
 //   q[t * q_ld + h * q_head_stride + c], out[t * out_ld + h * out_head_stride + c]; a cached key / value head starts every k_row / v_row
-//   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start).
+//   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start);
+//   q_group >= H / G: query head h lies in slot (h / (H / G)) q_group + h % (H / G) of its row;  gate (null, or [T, gate_ld] in the activation
+//   dtype, entry c of head h at h * dv + c): the output times the sigmoid of it.
 DSB_EXPORT int dsb200_sink_attention_ex(const void* q, long long q_ld, long long q_head_stride, const void* k_cache, long long k_block_stride, int k_row,
                                         const void* v_cache, long long v_block_stride, int v_row, const int* tok_seq, const int* tok_pos,
                                         const int* block_table, int bt_stride, int block_size, void* out, long long out_ld, long long out_head_stride,
                                         int n_tokens, int H, int G, int d, int dv, float scale, float cap, float sink, const float* sink_logit,
-                                        const float* r1, const float* r2, int part, int window, int dtype, cudaStream_t stream) {
+                                        const float* r1, const float* r2, int part, int window, int q_group, const void* gate, long long gate_ld, int dtype,
+                                        cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
   DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && d >= 1 && dv >= 1 && d + dv <= 8192 && sink >= 0.f && part >= 0 && window >= 0 && k_row >= d && v_row >= dv &&
-                  (r1 == nullptr) == (r2 == nullptr),
+                  (r1 != nullptr || r2 == nullptr) && q_group >= H / G && (gate == nullptr || gate_ld >= static_cast<long long>(H) * dv),
               "sink_attention: heads %d / %d, head sizes %d / %d, rows %d / %d, part %d", H, G, d, dv, k_row, v_row, part);
-  const SinkExtras ex{sink_logit, r1, r2, part, window, k_row, v_row, q_head_stride, out_head_stride};
+  const SinkExtras ex{sink_logit, r1, r2, part, window, k_row, v_row, q_head_stride, out_head_stride, q_group, gate, gate_ld};
   return launch_sink_attention(q, q_ld, k_cache, k_block_stride, v_cache, v_block_stride, tok_seq, tok_pos, block_table, bt_stride, block_size, out,
                                out_ld, n_tokens, H, G, d, dv, scale, cap, sink, ex, dtype, stream);
 }
 
 // Low-rank attention with one rotated key part shared by the heads.  proj [T, ld] (dtype 0 = bf16, 1 = fp32) holds per token the H query heads
 // (d plain entries, then dr entries to rotate) from q_col0 and the low-rank row (R entries, then dr entries to rotate) from kv_col0.  The
-// query heads' rotated parts are rotated IN PLACE (first rot_dims of the dr entries; entry i pairs with entry i + rot_dims / 2; angle =
-// pos * freq[i], freq: rot_dims / 2 doubles on the device); the first R entries of the low-rank row are RMS-normed with wkv [R] and, with the
+// query heads' rotated parts are rotated IN PLACE (first rot_dims of the dr entries; entry i pairs with entry i + rot_dims / 2, or -- interleaved --
+// entry 2i with entry 2i + 1; angle = pos * freq[i], freq: rot_dims / 2 doubles on the device); the first R entries of the low-rank row are RMS-normed with wkv [R] and, with the
 // rotated last dr entries behind them, written to the token's row of cache [blocks, block_size, row_w] (zeros from R + dr on).
 DSB_EXPORT int dsb200_latent_rotary_append(void* proj, long long ld, int q_col0, int kv_col0, const float* wkv, const double* freq, const int* tok_seq,
                                            const int* tok_pos, const int* block_table, int bt_stride, int block_size, void* cache, int row_w,
-                                           int n_tokens, int H, int d, int dr, int R, int rot_dims, float eps, int dtype, cudaStream_t stream) {
+                                           int n_tokens, int H, int d, int dr, int R, int rot_dims, float eps, int interleaved, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
   DSB_REQUIRE(H >= 1 && d >= 0 && dr >= 0 && R >= 1 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dr && (rot_dims == 0 || freq != nullptr) &&
                   row_w >= R + dr && wkv != nullptr,
@@ -588,10 +603,10 @@ DSB_EXPORT int dsb200_latent_rotary_append(void* proj, long long ld, int q_col0,
   const int grid = static_cast<int>((warps + wpb - 1) / wpb);
   if (dtype == 0)
     latent_rotary_append_kernel<bf16><<<grid, wpb * 32, 0, stream>>>((bf16*)proj, ld, q_col0, kv_col0, wkv, freq, tok_seq, tok_pos, block_table, bt_stride,
-                                                                    block_size, (bf16*)cache, row_w, n_tokens, H, d, dr, R, rot_dims, eps);
+                                                                    block_size, (bf16*)cache, row_w, n_tokens, H, d, dr, R, rot_dims, eps, interleaved);
   else
     latent_rotary_append_kernel<float><<<grid, wpb * 32, 0, stream>>>((float*)proj, ld, q_col0, kv_col0, wkv, freq, tok_seq, tok_pos, block_table,
-                                                                     bt_stride, block_size, (float*)cache, row_w, n_tokens, H, d, dr, R, rot_dims, eps);
+                                                                     bt_stride, block_size, (float*)cache, row_w, n_tokens, H, d, dr, R, rot_dims, eps, interleaved);
   DSB_CHECK_CUDA(cudaGetLastError());
   return DSB_OK;
 }
@@ -602,33 +617,34 @@ DSB_EXPORT int dsb200_latent_rotary_append(void* proj, long long ld, int q_col0,
 // rows of the sequence's earlier steps, WITHOUT the bias (update it afterwards with dsb200_conv_state_update).  Query / key heads: RMS norm over
 // d with wq / wk [d] shared by the heads -> q_out [T, q_ld] (head h at h * q_row) / the key plane.  Value heads: v_own (null, or [T, G dv])
 // receives the convolved values; with v_other ([T, G dv]) and mix (one float on the device) the cached value is (1 - mix) v + mix v_other.
-// Heads are padded with zeros to q_row / k_row / v_row entries.
+// Heads are padded with zeros to q_row / k_row / v_row entries.  wq / wk null: the norms have no weight.  q_group >= H / G: query head h goes to
+// slot (h / (H / G)) q_group + h % (H / G) of its row, slots without a head are zeros.  has_kv = 0: there are only queries (channels [H d]).
 DSB_EXPORT int dsb200_conv_head_norm_append(const void* proj, long long ld, int col0, const float* bias, const float* conv_w, const float* wq,
                                             const float* wk, const void* state, const int* seq_desc, const int* tok_seq, const int* tok_pos,
                                             const int* block_table, int bt_stride, int block_size, void* k_cache, long long k_block_stride,
                                             void* v_cache, long long v_block_stride, void* q_out, long long q_ld, const void* v_other,
                                             const float* mix, void* v_own, int n_tokens, int H, int G, int d, int dv, int taps, float eps, int q_row,
-                                            int k_row, int v_row, int dtype, cudaStream_t stream) {
+                                            int k_row, int v_row, int q_group, int has_kv, int dtype, cudaStream_t stream) {
   if (n_tokens == 0) return DSB_OK;
-  DSB_REQUIRE(H >= 1 && G >= 1 && d >= 1 && dv >= 1 && taps >= 1 && (taps == 1 || state != nullptr) && conv_w != nullptr && wq != nullptr &&
-                  wk != nullptr && (v_other == nullptr || mix != nullptr),
+  DSB_REQUIRE(H >= 1 && G >= 1 && H % G == 0 && q_group >= H / G && d >= 1 && dv >= 1 && taps >= 1 && (taps == 1 || state != nullptr) && conv_w != nullptr && (v_other == nullptr || mix != nullptr),
               "conv_head_norm_append: heads %d / %d, head sizes %d / %d, taps %d", H, G, d, dv, taps);
   DSB_REQUIRE(q_row >= d && k_row >= d && v_row >= dv, "conv_head_norm_append: row widths %d / %d / %d below the head sizes %d / %d", q_row, k_row, v_row, d, dv);
   auto mult4 = [](long long v) { return v % 4 == 0; };
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec = mult4(d) && mult4(dv) && mult4(ld) && mult4(col0) && mult4(q_ld) && mult4(q_row) && mult4(k_row) && mult4(v_row) && mult4(k_block_stride) &&
                    mult4(v_block_stride) && al16(proj) && al16(bias) && al16(conv_w) && al16(wq) && al16(wk) && al16(state) && al16(k_cache) && al16(v_cache) && al16(q_out) && al16(v_other) && al16(v_own);
+  const int per_tok = G * q_group + (has_kv ? 2 * G : 0);
   // several slots per warp when a lane's first group of channels covers a head and there are enough tokens to fill the GPU all the same
-  const bool many = (d > dv ? d : dv) <= (vec ? 128 : 32) && static_cast<long long>(n_tokens) * (H + 2 * G) >= 16384;
+  const bool many = (d > dv ? d : dv) <= (vec ? 128 : 32) && static_cast<long long>(n_tokens) * per_tok >= 16384;
   const int sl = many ? 4 : 1;
-  const long long warps = static_cast<long long>(n_tokens) * ((H + 2 * G + sl - 1) / sl);
+  const long long warps = static_cast<long long>(n_tokens) * ((per_tok + sl - 1) / sl);
   const int wpb = 8;
   const int grid = static_cast<int>((warps + wpb - 1) / wpb);
 #define LAUNCH(T, V, S)                                                                                                                                     \
   conv_head_norm_append_kernel<T, V, S><<<grid, wpb * 32, 0, stream>>>((const T*)proj, ld, col0, bias, conv_w, wq, wk, (const T*)state, (const int4*)seq_desc, tok_seq, \
                                                                        tok_pos, block_table, bt_stride, block_size, (T*)k_cache, k_block_stride, (T*)v_cache,         \
                                                                        v_block_stride, (T*)q_out, q_ld, (const T*)v_other, mix, (T*)v_own, n_tokens, H, G, d, dv,     \
-                                                                       taps, eps, q_row, k_row, v_row)
+                                                                       taps, eps, q_row, k_row, v_row, q_group, has_kv)
 #define PICK(T)                                                  \
   do {                                                           \
     if (vec && many) LAUNCH(T, 4, 4);                            \

@@ -231,7 +231,7 @@ native.register_sigs({
     "dsb200_sandwich_norm": "pp i p ff p f p i pp ii f i p",
     "dsb200_latent_norm_append": "p i pp pp ppp iiii ii f i p",
     "dsb200_paged_flash_latent": "p i ll pp ppp iiiiii f ii p i p",
-    "dsb200_paged_flash_latent_sink": "p i ll pp ppp iiiiii f p ii p i p",
+    "dsb200_paged_flash_latent_sink": "p i ll pp ppp iiiiii f p i ii p i p",
     "dsb200_gate_heads": "pp l p iii i p",
     "dsb200_latent_attention_scratch_floats": "iiii",
     "dsb200_latent_attention": "p i ll p i p ll p ppp ii iii f i p",
@@ -239,6 +239,7 @@ native.register_sigs({
     "dsb200_clamped_swish_gate": "pp l i fff i p",
     "dsb200_clamped_swish_gate_cols": "p l iii p l l i fff i p",
     "dsb200_stream_tanh_norm": "ppp i p ppp p i pp ii p",
+    "dsb200_gelu_gate_cols": "p l ii p l l i i p",
     "dsb200_softcap": "p l l i f p",
     "dsb200_grouped_topk_gating": "ppppppp iiiiiii p",
     "dsb200_moe_scatter_rows": "ppppppp iiii i p p",
@@ -348,14 +349,15 @@ def latent_norm_append(lat, wq, wkv, cache, tok_seq, tok_pos, block_table, nq, n
 
 
 def paged_latent_flash(q_abs, cache, tok_seq, tok_pos, block_table, scale, decode=False, max_context=None, n_splits=None, heads=None,
-                       sink_logit=None):
+                       sink_logit=None, window=0):
     """`latent_attention` on the tensor cores (csrc/attn/paged_flash.cu with one cache plane serving as keys and values).
     q_abs: bf16 view [T, H, rank] with unit stride in rank and any 16-byte-multiple token / head strides (token-major, or the
     head-major output of a batched GEMM seen through `.transpose(0, 1)`); rank 64 / 128.  The kernel works on `heads` heads, a divisor
     of 128 that is >= H (default: the next power of two); heads past H read as zero.  cache [blocks, block_size, rank] bf16 with a
     block size dividing 128.  Returns bf16 [T, heads, rank] (rows of heads >= H are meaningless).  `decode`: (almost) one token per
     sequence -- the small-atom kernel (rank 128, heads dividing 16).  `sink_logit` (fp32, one per head the kernel works on): learned sinks,
-    exp(sink_logit[h]) joins head h's softmax denominator."""
+    exp(sink_logit[h]) joins head h's softmax denominator.
+    `window` > 0: a query sees only the rows less than that far back (only their pages are visited)."""
     T, H, R = q_abs.shape
     Hp = heads or (1 << (H - 1).bit_length())
     assert sink_logit is None or (sink_logit.dtype == torch.float32 and sink_logit.numel() >= Hp and sink_logit.is_cuda)
@@ -365,7 +367,8 @@ def paged_latent_flash(q_abs, cache, tok_seq, tok_pos, block_table, scale, decod
     nt = (16 if decode else 128) // Hp
     max_atoms = max(1, min(T, (T + nt - 1) // nt + block_table.shape[0]))
     if n_splits is None:
-        pages = -(-(max_context if max_context is not None else block_table.shape[1] * bs) // 128)
+        ctx = max_context if max_context is not None else block_table.shape[1] * bs
+        pages = -(-(min(ctx, window + 256) if window > 0 else ctx) // 128)
         n_splits = _pick_splits(T, Hp, R, max_atoms, pages, page_us=0.45 if decode else 0.7)
     out = torch.empty(T, Hp, R, dtype=torch.bfloat16, device=q_abs.device)
     nbytes = native.lib().dsb200_paged_flash_scratch_bytes(T, Hp, R, max_atoms, n_splits)
@@ -373,7 +376,7 @@ def paged_latent_flash(q_abs, cache, tok_seq, tok_pos, block_table, scale, decod
     native.check(native.lib().dsb200_paged_flash_latent_sink(native.ptr(q_abs), H, q_abs.stride(1) if H > 1 else R, q_abs.stride(0) if T > 1 else H * R,
                                                              native.ptr(cache), native.ptr(out), native.ptr(tok_seq), native.ptr(tok_pos),
                                                              native.ptr(block_table), T, Hp, R, bs, block_table.shape[1], cache.shape[0], float(scale),
-                                                             native.ptr(sink_logit), max_atoms, n_splits, native.ptr(scratch), int(decode),
+                                                             native.ptr(sink_logit), int(window), max_atoms, n_splits, native.ptr(scratch), int(decode),
                                                              native.stream_ptr()), 2 + (n_splits > 1))
     return out
 
@@ -443,6 +446,15 @@ def clamped_swish_gate_cols(gu, gate_col0, up_col0, F, out, alpha, limit, shift,
     native.check(native.lib().dsb200_clamped_swish_gate_cols(native.ptr(gu), gu.stride(0), int(gate_col0), int(up_col0),
                                                              -1 if row_gate_col is None else int(row_gate_col), native.ptr(out), out.stride(0),
                                                              gu.shape[0], int(F), float(alpha), float(limit), float(shift), _dt(gu), native.stream_ptr()))
+    return out
+
+
+def gelu_gate_cols(gu, gate_col0, up_col0, F, out):
+    """gelu(gu[:, gate_col0 : gate_col0 + F]) * gu[:, up_col0 : up_col0 + F] (the tanh form of gelu) -> `out` [rows, F], a view with unit column
+    stride; forms and rounds like `clamped_swish_gate_cols` (accurate exponential in fp32)."""
+    assert gu.stride(1) == 1 and out.stride(1) == 1 and out.shape == (gu.shape[0], F) and gu.dtype == out.dtype
+    native.check(native.lib().dsb200_gelu_gate_cols(native.ptr(gu), gu.stride(0), int(gate_col0), int(up_col0), native.ptr(out), out.stride(0), gu.shape[0],
+                                                    int(F), _dt(gu), native.stream_ptr()))
     return out
 
 
@@ -527,7 +539,7 @@ native.register_sigs({
     "dsb200_head_norm_rotary_append": "p l iii pp p f ppp ii p l p l p l iiiii i f i iii ppp ii i p",
     "dsb200_sink_attention": "p l p l p l ppp ii p l iiiii fff i p",
     "dsb200_paged_flash_sink": "p l pp l ppp iiiiiii fff ii p i p",
-    "dsb200_paged_flash_sink_ex": "p l pp l ppp iiiiiii fff ppp ii ii p i p",
+    "dsb200_paged_flash_sink_ex": "p l pp l ppp iiiiiii fff ppp ii ii p l ii p i p",
 }, restype_long=("dsb200_scan_state_floats", ))
 
 
@@ -723,20 +735,22 @@ def sink_attention(q, k_plane, v_plane, tok_seq, tok_pos, block_table, block_siz
     return out
 
 
-def paged_flash_sink_ok(q, cache, out, H, G, d, dv):
+def paged_flash_sink_ok(q, cache, out, H, G, d, dv, compact=False):
     """Whether the tensor-core kernels take this attention: bf16, equal key / value head sizes of 64 / 128 in one two-plane cache tensor, a
-    q:kv head ratio dividing 128, cache blocks dividing 128, 16-byte aligned rows."""
+    q:kv head ratio dividing 128, cache blocks dividing 128, 16-byte aligned rows (of the queries alone for a `compact` output)."""
     return (q.is_cuda and q.dtype == torch.bfloat16 and cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and d == dv and d in (64, 128) and
             cache.dim() == 5 and H % G == 0 and 128 % (H // G) == 0 and cache.shape[2] >= 8 and 128 % cache.shape[2] == 0 and q.stride(0) % 8 == 0 and
-            out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0 and os.environ.get("DSB200_PAGED_FLASH", "1") != "0")
+            q.data_ptr() % 16 == 0 and (compact or (out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)) and os.environ.get("DSB200_PAGED_FLASH", "1") != "0")
 
 
 def paged_flash_sink(q, cache, tok_seq, tok_pos, block_table, out, H, G, d, scale, softcap=0.0, sink=1.0, decode=False, max_context=None, n_splits=None,
-                     sink_logit=None, r1=None, r2=None, part=0, window=0):
+                     sink_logit=None, r1=None, r2=None, part=0, window=0, compact=None, gate=None):
     """`sink_attention` / `sink_attention_ex` on the tensor cores (csrc/attn/paged_flash.cu: TMA pages through the block table, S / P / O in
     TMEM) for a two-plane cache [blocks, 2, block_size, G, d].  `decode`: (almost) one token per sequence -- the small-atom kernel.
     sink_logit / r1, r2 (fp32 [H]) / part: learned sinks, the logarithmic distance term and the mask by parts, as in `sink_attention_ex`;
-    `window` > 0: only the keys less than that far back (only their pages are visited)."""
+    `window` > 0: only the keys less than that far back (only their pages are visited).  `compact` (heads, entries): of every key / value head's
+    H / G query slots only the first `heads` are heads, and only the first `entries` of a head leave: out [T, G * heads * entries]; `gate` (a view
+    [T, G * heads * entries] of the activation dtype): the output times the sigmoid of it."""
     for p in (sink_logit, r1, r2):
         assert p is None or (p.dtype == torch.float32 and p.numel() == H and p.is_cuda)
     T = q.shape[0]
@@ -746,15 +760,18 @@ def paged_flash_sink(q, cache, tok_seq, tok_pos, block_table, out, H, G, d, scal
     max_atoms = max(1, min(T, (T + nt - 1) // nt + block_table.shape[0]))
     if n_splits is None:
         ctx = max_context if max_context is not None else block_table.shape[1] * bs
-        pages = -(-(min(ctx, window + 256) if window > 0 else ctx) // 128)
+        pages = -(-(min(ctx, window + 256) if window > 0 else (min(ctx, part + 128) if part > 0 else ctx)) // 128)
         n_splits = _pick_splits(T, H, d, max_atoms * G, pages, page_us=0.45 if decode else 0.7)
+    out_per, out_dv = compact if compact is not None else (0, 0)
+    assert gate is None or (compact is not None and gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (T, G * out_per * out_dv))
     nbytes = native.lib().dsb200_paged_flash_scratch_bytes(T, H, d, max_atoms, n_splits)
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
     native.check(native.lib().dsb200_paged_flash_sink_ex(native.ptr(q), q.stride(0), native.ptr(cache), native.ptr(out), out.stride(0), native.ptr(tok_seq),
                                                          native.ptr(tok_pos), native.ptr(block_table), T, H, G, d, bs, block_table.shape[1],
                                                          cache.shape[0], float(scale), float(softcap), float(sink), native.ptr(sink_logit),
-                                                         native.ptr(r1), native.ptr(r2), int(part), int(window), max_atoms, n_splits, native.ptr(scratch),
-                                                         int(decode), native.stream_ptr()), 2 + (n_splits > 1))
+                                                         native.ptr(r1), native.ptr(r2), int(part), int(window), int(out_dv), int(out_per),
+                                                         native.ptr(gate), gate.stride(0) if gate is not None else 0, max_atoms, n_splits,
+                                                         native.ptr(scratch), int(decode), native.stream_ptr()), 2 + (n_splits > 1))
     return out
 
 
@@ -767,9 +784,9 @@ native.register_sigs({
     "dsb200_gate_heads_scalar": "pp l p l iii i p",
     "dsb200_mingru_scratch_floats": "iii",
     "dsb200_mingru_scan": "p l iii pp pp p p l iii i p i p",
-    "dsb200_sink_attention_ex": "p l l p l i p l i ppp ii p l l iiiii fff ppp ii i p",
-    "dsb200_latent_rotary_append": "p l ii pp ppp ii p i iiiii i f i p",
-    "dsb200_conv_head_norm_append": "p l i pppp p pppp ii p l p l p l p p p iiiiii f iii i p",
+    "dsb200_sink_attention_ex": "p l l p l i p l i ppp ii p l l iiiii fff ppp ii i p l i p",
+    "dsb200_latent_rotary_append": "p l ii pp ppp ii p i iiiii i f i i p",
+    "dsb200_conv_head_norm_append": "p l i pppp p pppp ii p l p l p l p p p iiiiii f iii ii i p",
 }, restype_long=("dsb200_mingru_scratch_floats", ))
 
 
@@ -836,55 +853,63 @@ def mingru_scan(proj, z_col0, x_col0, g_col0, z_bias, x_bias, tok_seq, seq_desc,
 
 
 def sink_attention_ex(q, q_head_stride, k_plane, k_row, v_plane, v_row, tok_seq, tok_pos, block_table, block_size, out, out_head_stride, H, G, d, dv,
-                      scale, softcap=0.0, sink=0.0, sink_logit=None, r1=None, r2=None, part=0, window=0):
+                      scale, softcap=0.0, sink=0.0, sink_logit=None, r1=None, r2=None, part=0, window=0, q_group=None, gate=None):
     """`sink_attention` with learned sinks (sink_logit fp32 [H]: exp of it joins the head's denominator), a distance term (r1, r2 fp32 [H]: the
-    score of key j loses r1 ln(1 + r2 (pos - j))), a mask by parts (`part` > 0: a query sees only the keys of its own part of that many
+    score of key j loses r1 ln(1 + r2 (pos - j)); r1 alone: r1 (pos - j)), a mask by parts (`part` > 0: a query sees only the keys of its own part of that many
     positions, counted from the sequence's start), a sliding window (`window` > 0: only keys less than that far back) and free strides: q / out are addressed [t * stride(0) + h * head_stride + c], a cached
-    key / value head starts every k_row / v_row elements of its token's row."""
+    key / value head starts every k_row / v_row elements of its token's row.  `q_group` (>= H / G): slots per key / value head in a query row.  `gate`
+    (a view [T, H dv] of the activation dtype): entry c of head h is multiplied by the sigmoid of gate[:, h dv + c]."""
     T = q.shape[0]
     (kc, ks), (vc, vs) = k_plane, v_plane
     assert q.dtype == kc.dtype == vc.dtype == out.dtype
     for p in (sink_logit, r1, r2):
         assert p is None or (p.dtype == torch.float32 and p.numel() == H and p.is_cuda)
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (T, H * dv))
     native.check(native.lib().dsb200_sink_attention_ex(native.ptr(q), q.stride(0), int(q_head_stride), native.ptr(kc), ks, int(k_row), native.ptr(vc), vs,
                                                        int(v_row), native.ptr(tok_seq), native.ptr(tok_pos), native.ptr(block_table),
                                                        block_table.stride(0), int(block_size), native.ptr(out), out.stride(0), int(out_head_stride), T,
                                                        H, G, d, dv, float(scale), float(softcap), float(sink), native.ptr(sink_logit), native.ptr(r1),
-                                                       native.ptr(r2), int(part), int(window), _dt(q), native.stream_ptr()))
+                                                       native.ptr(r2), int(part), int(window), int(q_group or H // G), native.ptr(gate),
+                                                       gate.stride(0) if gate is not None else 0, _dt(q), native.stream_ptr()))
     return out
 
 
-def latent_rotary_append(proj, q_col0, kv_col0, wkv, freq, tok_seq, tok_pos, block_table, cache, H, d, dr, R, rot_dims, eps):
+def latent_rotary_append(proj, q_col0, kv_col0, wkv, freq, tok_seq, tok_pos, block_table, cache, H, d, dr, R, rot_dims, eps, interleaved=False):
     """proj [T, N] holds the H query heads (d plain + dr rotated entries each) from q_col0 and the low-rank row (R + dr entries) from kv_col0.
-    The rotated parts of the query heads are rotated in place (rotate-half pairs over the first rot_dims of the dr entries, angle pos * freq[i]);
+    The rotated parts of the query heads are rotated in place (pairs (i, i + rot_dims / 2) -- `interleaved`: (2i, 2i + 1) -- over the first rot_dims
+    of the dr entries, angle pos * freq[i]);
     the RMS-normed (weight wkv) first R entries of the low-rank row and its rotated last dr entries go to the token's row of
     cache [blocks, block_size, row >= R + dr] (zeros behind)."""
     assert proj.stride(1) == 1 and cache.is_contiguous() and cache.dim() == 3 and cache.dtype == proj.dtype
     native.check(native.lib().dsb200_latent_rotary_append(native.ptr(proj), proj.stride(0), q_col0, kv_col0, native.ptr(wkv), native.ptr(freq),
                                                           native.ptr(tok_seq), native.ptr(tok_pos), native.ptr(block_table), block_table.stride(0),
                                                           cache.shape[1], native.ptr(cache), cache.shape[2], proj.shape[0], H, d, dr, R, int(rot_dims),
-                                                          float(eps), _dt(proj), native.stream_ptr()))
+                                                          float(eps), int(interleaved), _dt(proj), native.stream_ptr()))
 
 
 def conv_head_norm_append(proj, col0, bias, conv_w, wq, wk, state, seq_desc, tok_seq, tok_pos, block_table, block_size, k_plane, v_plane, q_out,
-                          H, G, d, dv, taps, eps, v_other=None, mix=None, v_own=None, row=None):
+                          H, G, d, dv, taps, eps, v_other=None, mix=None, v_own=None, row=None, q_group=None, kv=True):
     """Query heads [H d], key heads [G d] and value heads [G dv] lie side by side in proj from column col0.  Every channel gets its bias
     (fp32, or None) and a short causal convolution (conv_w fp32 [taps, channels]; rows before this step's come from state
     [slots, taps - 1, channels], rows before the sequence are zeros); query / key heads are RMS-normed with wq / wk [d] (shared by the heads);
     queries -> q_out, keys / values -> their planes.  v_own ([T, G dv]): receives the convolved values; v_other + mix (fp32 [1]): the cached
-    value is (1 - mix) v + mix v_other.  `row`: heads are padded with zeros to this width."""
-    (kc, ks), (vc, vs) = k_plane, v_plane
-    assert proj.stride(1) == 1 and q_out.stride(1) == 1 and q_out.dtype == proj.dtype == kc.dtype == vc.dtype
+    value is (1 - mix) v + mix v_other.  `row`: heads are padded with zeros to this width.  wq / wk None: norms without a weight.  `q_group` (>= H /
+    G): slots per key / value head in a query row (zeros in the slots without a head).  `kv` False: there are only queries (channels [H d]); the
+    planes are left alone and may be None."""
+    (kc, ks), (vc, vs) = (k_plane, v_plane) if kv else ((None, 0), (None, 0))
+    assert proj.stride(1) == 1 and q_out.stride(1) == 1 and q_out.dtype == proj.dtype and (not kv or kc.dtype == vc.dtype == proj.dtype)
     for v in (v_other, v_own):
         assert v is None or (v.is_contiguous() and v.dtype == proj.dtype and v.shape == (proj.shape[0], G * dv))
     assert state is None or (state.dtype == proj.dtype and state.is_contiguous())
-    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape == (taps, (H + G) * d + G * dv)
+    assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape == (taps, H * d + (G * (d + dv) if kv else 0))
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == conv_w.shape[1])
     native.check(native.lib().dsb200_conv_head_norm_append(native.ptr(proj), proj.stride(0), col0, native.ptr(bias), native.ptr(conv_w), native.ptr(wq),
                                                            native.ptr(wk), native.ptr(state), native.ptr(seq_desc), native.ptr(tok_seq),
                                                            native.ptr(tok_pos), native.ptr(block_table), block_table.stride(0), int(block_size),
                                                            native.ptr(kc), ks, native.ptr(vc), vs, native.ptr(q_out), q_out.stride(0),
                                                            native.ptr(v_other), native.ptr(mix), native.ptr(v_own), proj.shape[0], H, G, d, dv, int(taps),
-                                                           float(eps), int(row or d), int(row or d), int(row or dv), _dt(proj), native.stream_ptr()))
+                                                           float(eps), int(row or d), int(row or d), int(row or dv), int(q_group or H // G), int(kv), _dt(proj),
+                                                           native.stream_ptr()))
     return q_out
 
 
@@ -967,3 +992,33 @@ def gated_group_norm(y, z, w, out, groups, eps):
     native.check(native.lib().dsb200_gated_group_norm(native.ptr(y), native.ptr(z), z.stride(0), native.ptr(w), native.ptr(out), out.stride(0), T, inner,
                                                       int(groups), float(eps), _dt(z), native.stream_ptr()))
     return out
+
+
+# ---- kernels of csrc/ragged/hyper_ops.cu: residuals made of several parallel streams
+native.register_sigs({"dsb200_stream_mix_norm": "p i p p l i pp pp pp p i p l ii f p"})
+
+
+def stream_mix_norm(x, n_streams, branch=None, w_in=None, gamma=None, eps=1e-6, out_dtype=torch.bfloat16, rows=None):
+    """x fp32: the residual streams [T, n_streams, dim], or [T, dim] when all of them are (still) equal.  `branch` = (y, bias, scale, mix, w_out), the
+    finished sublayer's output y [T, dim] (activation dtype; bias / scale fp32 [dim] or None): every stream t becomes
+    sum_s mix[s, t] x_s + w_out[t] scale (y + bias).  With gamma: the sum of the (joined) streams weighted with w_in (None: ones), RMS-normed, times
+    gamma, in `out_dtype`.  Returns (streams, normed or None): the streams are x itself, updated in place (a new tensor when x was one row for all
+    of them).  `rows` (int32 indices): join and norm only those rows, for the normed result alone; x is left as it was."""
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.is_cuda and (x.dim() == 2 or x.shape[1] == n_streams)
+    T, dim, shared = x.shape[0], x.shape[-1], x.dim() == 2
+    y, bias, scale, mix, w_out = branch if branch is not None else (None, ) * 5
+    for p, k in ((bias, dim), (scale, dim), (mix, n_streams * n_streams), (w_out, n_streams), (w_in, n_streams), (gamma, dim)):
+        assert p is None or (p.dtype == torch.float32 and p.is_cuda and p.is_contiguous() and p.numel() == k)
+    assert y is None or (y.shape == (T, dim) and y.stride(1) == 1 and mix is not None and w_out is not None)
+    x_out = None
+    if y is not None and rows is None:
+        x_out = torch.empty(T, n_streams, dim, dtype=torch.float32, device=x.device) if shared else x
+    n = T if rows is None else rows.numel()
+    out = torch.empty(n, dim, dtype=out_dtype, device=x.device) if gamma is not None else None
+    if out is None and x_out is None:
+        return x, None
+    native.check(native.lib().dsb200_stream_mix_norm(native.ptr(x), int(shared), native.ptr(x_out), native.ptr(y), y.stride(0) if y is not None else 0,
+                                                     _dt(y) if y is not None else 0, native.ptr(bias), native.ptr(scale), native.ptr(mix),
+                                                     native.ptr(w_out), native.ptr(w_in), native.ptr(gamma), native.ptr(out), _DT[out_dtype],
+                                                     native.ptr(rows), n, int(n_streams), dim, float(eps), native.stream_ptr()))
+    return (x if x_out is None else x_out), out

@@ -188,8 +188,8 @@ class DSSinkAttentionConfig(DSModuleConfig):
 class DSRotaryLatentAttentionConfig(DSModuleConfig):
     """Attention whose keys and values are per-head up-projections of one cached, RMS-normed low-rank latent per token, with a rotated part
     beside it: a query head has `qk_dim` plain and `rot_dim` rotated entries; every token adds ONE rotated key part of `rot_dim` entries that
-    all heads share, cached beside the latent.  score = scale (q_plain . W_uk c + q_rot . k_rot); rotate-half pairs over the first `rotate_dim`
-    of the rot_dim entries; causal softmax, optionally with a learned sink per head (exp(sink_h) joins the denominator) and a sigmoid gate
+    all heads share, cached beside the latent.  score = scale (q_plain . W_uk c + q_rot . k_rot); rotate-half pairs (`interleaved`: neighbouring
+    entries are paired) over the first `rotate_dim` of the rot_dim entries; causal softmax, optionally over a sliding `window` and with a learned sink per head (exp(sink_h) joins the denominator) and a sigmoid gate
     per token and head on the head's output."""
     n_heads: int
     qk_dim: int  # plain (unrotated) query / key entries per head
@@ -198,7 +198,9 @@ class DSRotaryLatentAttentionConfig(DSModuleConfig):
     kv_rank: int
     scale: float
     rotate_dim: int  # entries of the rot_dim part that are rotated (pairs (i, i + rotate_dim / 2)); the rest pass unchanged
+    interleaved: bool = False  # pairs are (2i, 2i + 1) instead
     theta_base: float = 10_000.0
+    window: int = 0  # > 0: a query sees only the keys less than this far back (itself and the window - 1 tokens before it)
     learned_sink: bool = False
     head_gate: bool = False
     eps: float = 1e-6  # of the latent's norm
@@ -215,6 +217,8 @@ class DSRotaryLatentAttentionConfig(DSModuleConfig):
             raise ValueError("a query head needs at least one entry")
         if not (0 <= self.rotate_dim <= self.rot_dim and self.rotate_dim % 2 == 0):
             raise ValueError(f"rotate_dim must be even and at most rot_dim ({self.rot_dim}), got {self.rotate_dim}")
+        if self.window < 0:
+            raise ValueError(f"window cannot be negative, got {self.window}")
         if self.kv_rank + self.rot_dim > 4096:
             raise ValueError("the attention kernels hold a cached row of at most 4096 values")
         return self
@@ -222,10 +226,12 @@ class DSRotaryLatentAttentionConfig(DSModuleConfig):
 
 class DSConvSinkAttentionConfig(DSModuleConfig):
     """Attention whose query, key and value projections (with biases) pass a short causal convolution over time, then per-head RMS norms of
-    queries and keys (one weight of head size shared by the heads); no rotation.  score = scale q . k - r1_h ln(1 + r2_h (i - j)) when
-    `distance_bias`; a query at position i sees the keys j <= i of its own part, floor(i / part_size) = floor(j / part_size) (0: all);
+    queries and keys (one weight of head size shared by the heads, none with `qk_norm_weight` off); no rotation.  score = scale q . k
+    - r1_h ln(1 + r2_h (i - j)) when `distance_bias`, - 2^(-8 (h + 1) / heads) (i - j) when `linear_bias`; a query at position i sees the keys j <= i of its own part, floor(i / part_size) = floor(j / part_size) (0: all);
     `learned_sink`: exp(sink_h) joins the softmax denominator.  `value_mix`: "source" = the layer's convolved values are handed to later
-    layers; "mix" = the cached value is (1 - m) v + m v_source with the source layer's values of the same token; "none"."""
+    layers; "mix" = the cached value is (1 - m) v + m v_source with the source layer's values of the same token; "none".  `output_gate`: the
+    concatenated heads are multiplied by the sigmoid of pre-activations handed to the module; `reads_cache`: the layer has queries only and reads the
+    keys and values that another layer of equal key / value heads wrote to ITS cache."""
     n_heads_q: int
     n_heads_kv: int
     head_size: int
@@ -233,9 +239,13 @@ class DSConvSinkAttentionConfig(DSModuleConfig):
     conv_taps: int  # the last taps - 1 projected rows of a sequence are state
     scale: float
     part_size: int = 0
+    qk_norm_weight: bool = True
     distance_bias: bool = False
+    linear_bias: bool = False
     learned_sink: bool = False
     value_mix: str = "none"
+    output_gate: bool = False
+    reads_cache: bool = False
     eps: float = 1e-6
     max_sequences: int
     input_dtype: DtypeEnum = DtypeEnum.bf16
@@ -249,6 +259,10 @@ class DSConvSinkAttentionConfig(DSModuleConfig):
             raise ValueError("head sizes and conv_taps must be positive, part_size cannot be negative")
         if self.value_mix not in ("none", "source", "mix"):
             raise ValueError(f"value_mix must be none, source or mix, got {self.value_mix}")
+        if self.distance_bias and self.linear_bias:
+            raise ValueError("a score has one distance term")
+        if self.reads_cache and self.value_mix != "none":
+            raise ValueError("a layer without values of its own cannot mix them")
         return self
 
     @property

@@ -30,6 +30,9 @@ class DSNormConfig(DSModuleConfig):
     # The sublayers read the stream itself; the stream is kept in fp32 and handed on in the activation dtype as well.
     post_sum: bool = False
     stream_mult: float = 1.0
+    # "hyper-connection" blocks (> 0): the residual is this many parallel fp32 streams; the norm reads a weighted sum of them, and a sublayer's
+    # output (times a weight per channel) joins all of them while they are mixed with one another.
+    streams: int = 0
 
     @field_validator("channels")
     @classmethod

@@ -16,4 +16,5 @@ class DSUnembedConfig(DSModuleConfig):
     logit_softcap: float = 0.0  # > 0: logits <- cap * tanh(logits / cap)
     residual_fp32: bool = False  # the hidden states arrive as the fp32 residual stream; logits leave in fp32
     logit_scale: float = 1.0  # the logits are multiplied by this (folded into the final norm's weight: `transform_norm_param`)
+    streams: int = 0  # > 0, with residual_fp32: the residual is this many parallel streams, whose sum is normed
     norm_groups: int = 1  # with residual_fp32: the final RMS norm works on this many equal consecutive parts of the row, each on its own

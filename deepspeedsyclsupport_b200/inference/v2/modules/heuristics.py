@@ -23,7 +23,7 @@ def instantiate_attention(attention_config, engine_config: RaggedInferenceEngine
         return DSSelfAttentionRegistry.instantiate_config(ConfigBundle(name="latent_blocked_attention", config=attention_config))
     if isinstance(attention_config, DSRotaryLatentAttentionConfig):  # a cached latent with one rotated key part beside it, learned sinks
         return DSSelfAttentionRegistry.instantiate_config(ConfigBundle(name="rotary_latent_attention", config=attention_config))
-    if isinstance(attention_config, DSConvSinkAttentionConfig):  # convolved q / k / v, distance term, mask by parts, learned sinks, value mixing
+    if isinstance(attention_config, DSConvSinkAttentionConfig):  # convolved q / k / v, distance terms, mask by parts, learned sinks, value mixing, output gate
         return DSSelfAttentionRegistry.instantiate_config(ConfigBundle(name="conv_sink_attention", config=attention_config))
     if isinstance(attention_config, DSWindowedAttentionConfig):  # convolved q / k, values = keys, sliding window that keeps the first tokens
         return DSSelfAttentionRegistry.instantiate_config(ConfigBundle(name="windowed_conv_attention", config=attention_config))
@@ -75,6 +75,8 @@ def instantiate_pre_norm(norm_config: DSNormConfig, engine_config: RaggedInferen
     name = "cuda_pre_ln" if kind == NormTypeEnum.LayerNorm else ("cuda_sandwich_rms" if norm_config.sandwich else "cuda_pre_rms")
     if kind == NormTypeEnum.RMSNorm and norm_config.shared_input:
         name = "cuda_group_rms"
+    elif kind == NormTypeEnum.RMSNorm and norm_config.streams > 0:
+        name = "cuda_stream_mix_rms"
     elif kind == NormTypeEnum.DynamicTanh:
         name = "cuda_dynamic_tanh"
     return DSPreNormRegistry.instantiate_config(ConfigBundle(name=name, config=norm_config))

@@ -26,21 +26,21 @@ from ...configs import DSLatentAttentionConfig
 from ...interfaces import DSSelfAttentionBase, DSSelfAttentionRegistry
 
 
-def _bmm(a, b, out_dtype):
-    """Batched a @ b with fp32 accumulation; fp32 operands in true fp32."""
+def _bmm(a, b, out_dtype, out=None):
+    """Batched a @ b with fp32 accumulation; fp32 operands in true fp32.  `out`: a tensor (any strides) of the operands' dtype for the result."""
     if a.dtype == torch.float32:
         keep = torch.backends.cuda.matmul.allow_tf32
         torch.backends.cuda.matmul.allow_tf32 = False
         try:
-            return torch.bmm(a, b)
+            return torch.bmm(a, b, out=out)
         finally:
             torch.backends.cuda.matmul.allow_tf32 = keep
-    if out_dtype == torch.float32:
+    if out_dtype == torch.float32 and out is None:
         try:
             return torch.bmm(a, b, out_dtype=torch.float32)
         except (TypeError, RuntimeError):
             return torch.bmm(a, b).float()
-    return torch.bmm(a, b)
+    return torch.bmm(a, b, out=out)
 
 
 @DSSelfAttentionRegistry.register_module

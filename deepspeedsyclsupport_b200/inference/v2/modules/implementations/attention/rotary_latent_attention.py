@@ -7,9 +7,11 @@ into the latent space once per token (a batched GEMM whose right operand also ca
 of a token then share the cached rows as keys, their first kv_rank values as values, and the value up-projection is applied to the attended
 latent.  Nothing but the row is cached or expanded, for prompt portions and decode steps alike.
 
+The mask may be a sliding window; pairs of rotated entries are (i, i + n / 2) or neighbours.
+
 Per layer: rotation of the query heads' rotated parts in place + latent norm + key rotation + cache append (one kernel), per-head map into the
-latent space (batched GEMM), the attention kernel with a learned sink per head, per-head value up-projection (batched GEMM), head
-concatenation + sigmoid gate per (token, head) in one pass.
+latent space (batched GEMM), the attention kernel, optionally with a learned sink per head, per-head value up-projection (batched GEMM, which
+leaves the heads side by side per token), or with the sigmoid gate per (token, head): head concatenation + gate in one pass.
 
 Two attention kernels.  bf16 with kv_rank + rot_dim <= 128 and at most 128 heads: the tcgen05 paged flash kernels in their one-plane mode with
 per-head sinks (rows zero-padded to 64 / 128 values, heads to a divisor of 128: neither changes a score or an output).  Everything else:
@@ -112,34 +114,33 @@ class DSRotaryLatentAttention(DSSelfAttentionBase):
         low-rank row (kv_rank | rot_dim) at cols[1] and, with `head_gate`, one gate pre-activation per head at cols[2]; the query heads'
         rotated parts are overwritten.  kv_cache [blocks, block_size, 1, row].  sink fp32 [heads].  Returns [T, heads * v_dim]."""
         c = self._config
-        q0, kv0, g0 = cols
+        q0, kv0, g0 = cols if c.head_gate else (*cols[:2], None)
         T, H, R, dq = proj.shape[0], c.n_heads, self._row, c.qk_dim + c.rot_dim
         cache = kv_cache.view(kv_cache.shape[0], kv_cache.shape[1], R)
         tok_seq, tok_pos, bt = batch.tok_seq(), batch.tok_pos(), batch.block_table()
         if c.rotate_dim and (self._freq is None or self._freq.device != proj.device):
             self._freq = self._freq_host.to(proj.device)
         K.latent_rotary_append(proj, q0, kv0, kv_norm_w, self._freq if c.rotate_dim else None, tok_seq, tok_pos, bt, cache, H, c.qk_dim, c.rot_dim,
-                               c.kv_rank, c.rotate_dim, c.eps)
+                               c.kv_rank, c.rotate_dim, c.eps, interleaved=c.interleaved)
         q = proj[:, q0:q0 + H * dq].view(T, H, dq).transpose(0, 1)  # [H, T, dq]
         bs = cache.shape[1]
         sink = sink if c.learned_sink else None
         if self._flash and bs >= 8 and 128 % bs == 0:
             qa = torch.bmm(q, key_up_w)  # [H, T, R]; the kernel reads it head-major through its TMA strides, missing heads as zeros
-            att = K.paged_latent_flash(qa.transpose(0, 1), cache, tok_seq, tok_pos, bt, c.scale, heads=self._heads_p, sink_logit=sink,
+            att = K.paged_latent_flash(qa.transpose(0, 1), cache, tok_seq, tok_pos, bt, c.scale, heads=self._heads_p, sink_logit=sink, window=c.window,
                                        decode=batch.current_tokens <= 2 * batch.current_sequences)
-            o = torch.bmm(att[:, :H].transpose(0, 1), value_up_w)  # [H, T, v_dim]
+            att = att[:, :H].transpose(0, 1)
         else:
             qa = _bmm(q, key_up_w, self._dtype)  # [H, T, R]
             W = self.attended_width
             att = torch.empty(H, T, W, dtype=self._dtype, device=proj.device)
             plane = (cache, cache.stride(0))
             K.sink_attention_ex(qa.transpose(0, 1), qa.stride(0), plane, R, plane, R, tok_seq, tok_pos, bt, bs, att.transpose(0, 1), att.stride(0), H, 1,
-                                R, W, c.scale, sink_logit=sink[:H] if sink is not None else None)
-            o = _bmm(att, value_up_w, self._dtype)  # [H, T, v_dim]
+                                R, W, c.scale, sink_logit=sink[:H] if sink is not None else None, window=c.window)
         if c.head_gate:
+            o = _bmm(att, value_up_w, self._dtype)  # [H, T, v_dim]
             return K.gate_heads_scalar(o.contiguous(), proj[:, g0:g0 + H], out)  # heads side by side per token and the gate, one pass
-        o = o.transpose(0, 1).reshape(T, H * c.v_dim)
-        if out is not None:
-            out.copy_(o)
-            return out
-        return o
+        if out is None:
+            out = torch.empty(T, H * c.v_dim, dtype=self._dtype, device=proj.device)
+        _bmm(att, value_up_w, self._dtype, out=out.view(T, H, c.v_dim).transpose(0, 1))  # the GEMM's strides put the heads side by side
+        return out

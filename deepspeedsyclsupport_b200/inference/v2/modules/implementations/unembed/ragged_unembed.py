@@ -41,7 +41,7 @@ class DSRaggedUnembed(DSUnembedBase):
         """`residual` (optional): the residual stream the last hidden state still has to be added to -- only the gathered rows
         (one per sequence) are added and normalised, not the whole batch.  `pending` (fp32 stream only): ((outputs in the activation
         dtype, ...), fp32 output or None) of the last layer's sublayers that have not joined the stream yet; they are added to the
-        gathered rows only."""
+        gathered rows only; with `streams` it is one sublayer's branch as `kernels.stream_mix_norm` takes it."""
         last_tok = ragged_metadata.logit_rows()
         c = self._config
         if c.residual_fp32:
@@ -68,14 +68,16 @@ class DSRaggedUnembed(DSUnembedBase):
         return logits
 
     def _forward_fp32_residual(self, residual, vocab_embedding, rows, gamma, pending=None, beta=None, alpha=None):
-        """Gather + RMS norm (or tanh(alpha x) * gamma + beta) of the wanted rows in one kernel (fp32 in, activation dtype out), projection with fp32 logits,
-        soft cap in place."""
+        """Gather + RMS norm (or tanh(alpha x) * gamma + beta) of the wanted rows, or of the sum of their streams, in one kernel (fp32 in, activation
+        dtype out), projection with fp32 logits, soft cap in place."""
         c = self._config
         assert self._norm in (NormTypeEnum.RMSNorm, NormTypeEnum.DynamicTanh) and residual.dtype == torch.float32
         act = DtypeEnum(c.dtype).value
         if rows.numel() == 0:
             return torch.empty(0, vocab_embedding.shape[0], dtype=torch.float32, device=residual.device)
-        if self._norm == NormTypeEnum.DynamicTanh:
+        if c.streams > 0:
+            h = K.stream_mix_norm(residual, c.streams, pending, None, gamma, c.eps, out_dtype=act, rows=rows)[1]
+        elif self._norm == NormTypeEnum.DynamicTanh:
             branches, fp32_branch = pending if pending is not None else ((), None)
             h = K.stream_tanh_norm(residual, branches, fp32_branch, alpha, gamma, beta, out_dtype=act, rows=rows)
         elif c.norm_groups > 1 or pending is not None:  # the stream still lacks the last layer's outputs and / or is normed in parts

@@ -151,12 +151,14 @@ int dsb200_paged_flash_decode(const void* qkv, const void* kv_cache, void* out, 
  * head-major [heads][T][rank]); the kernel works on `heads` heads (a divisor of 128), the ones past q_heads read as zero.
  * out is [n_tokens][heads][rank] bf16; rank 64 or 128.  decode != 0 selects the small-atom kernel (rank 128, heads dividing 16).
  * Scratch and atoms as for dsb200_paged_flash_attention with hq = heads.
- * sink_logit (null, or `heads` floats): exp(sink_logit[h]) joins head h's softmax denominator, an entry without key and value. */
+ * sink_logit (null, or `heads` floats): exp(sink_logit[h]) joins head h's softmax denominator, an entry without key and value.
+ * window > 0: a query at position i sees only the rows with i - j < window (only their pages are visited); 0 = the whole history. */
 int dsb200_paged_flash_latent_sink(const void* q, int q_heads, long long q_head_stride, long long q_tok_stride,
                                    const void* cache, void* out, const int* tok_seq, const int* tok_pos,
                                    const int* block_table, int n_tokens, int heads, int rank, int block_size,
                                    int max_blocks_per_seq, int num_blocks, float scale, const float* sink_logit,
-                                   int max_atoms, int n_splits, void* scratch, int decode, dsb200_stream_t stream);
+                                   int window, int max_atoms, int n_splits, void* scratch, int decode,
+                                   dsb200_stream_t stream);
 int dsb200_paged_flash_latent(const void* q, int q_heads, long long q_head_stride, long long q_tok_stride,
                               const void* cache, void* out, const int* tok_seq, const int* tok_pos, const int* block_table,
                               int n_tokens, int heads, int rank, int block_size, int max_blocks_per_seq, int num_blocks,
@@ -176,14 +178,16 @@ int dsb200_paged_flash_window(const void* q, long long q_tok_stride, const void*
  * bf16 at q_tok_stride elements per token (a multiple of 8), kv_cache [num_blocks][2][block_size][hkv][head_dim] bf16; out rows at out_ld
  * elements per token (a multiple of 8).  decode != 0 selects the small-atom kernel (head_dim 128, q:kv head ratios dividing 16).
  * sink_logit (hq floats): learned sinks, exp(sink_logit[h]) joins head h's denominator; r1, r2 (hq floats each): the score of key j for the
- * query at position i loses r1[h] ln(1 + r2[h] (i - j)); part > 0: a query sees only the keys of its own part of `part` positions;
- * window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0). */
+ * query at position i loses r1[h] ln(1 + r2[h] (i - j)), r1 alone: it loses r1[h] (i - j); part > 0: a query sees only the keys of its own part of
+ * `part` positions; window > 0: a query at position i sees only the keys with i - j < window (not together with part).  Each may be absent (null / 0).
+ * out_dv > 0: compact output -- of every group of hq / hkv slots only the first out_per are heads, and only the first out_dv entries of a head leave:
+ * out row [hkv * out_per][out_dv]; gate (null, or bf16 [n_tokens][gate_ld] in that layout): the output times the sigmoid of it. */
 int dsb200_paged_flash_sink_ex(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld,
                                const int* tok_seq, const int* tok_pos, const int* block_table, int n_tokens, int hq,
                                int hkv, int head_dim, int block_size, int max_blocks_per_seq, int num_blocks, float scale,
                                float softcap, float sink, const float* sink_logit, const float* r1, const float* r2,
-                               int part, int window, int max_atoms, int n_splits, void* scratch, int decode,
-                               dsb200_stream_t stream);
+                               int part, int window, int out_dv, int out_per, const void* gate, long long gate_ld,
+                               int max_atoms, int n_splits, void* scratch, int decode, dsb200_stream_t stream);
 int dsb200_paged_flash_sink(const void* q, long long q_tok_stride, const void* kv_cache, void* out, long long out_ld,
                             const int* tok_seq, const int* tok_pos, const int* block_table, int n_tokens, int hq, int hkv,
                             int head_dim, int block_size, int max_blocks_per_seq, int num_blocks, float scale,
@@ -400,6 +404,17 @@ int dsb200_fake_quantize(void* x, long long groups, int group_size, int bits, in
 int dsb200_fp8_rowwise_quantize(const void* x, void* q, float* scales, int rows, int cols, long long ldx, int dtype,
                                 dsb200_stream_t stream);
 
+/* ---- csrc/ragged/hyper_ops.cu */
+/* x fp32: the streams [T, S, dim], or (shared_row) one row [T, dim] that stands for all of them.  y (null: no join) [T, y_ld] in y_dtype (0 =
+ * bf16, 1 = fp32): the finished sublayer's output; bias, scale [dim] fp32 or null; mix [S, S] (from, to), w_out [S].  The joined streams go to
+ * x_out [T, S, dim] (x itself unless shared_row; null: nowhere).  gamma (null: nothing is read) [dim]: out [n, dim] in out_dtype receives the
+ * RMS-normed sum of the streams weighted with w_in [S] (null: ones).  rows (null, or n int32 token rows): only these rows are worked on; x_out
+ * must then be null. */
+int dsb200_stream_mix_norm(const float* x, int shared_row, float* x_out, const void* y, long long y_ld, int y_dtype,
+                           const float* bias, const float* scale, const float* mix, const float* w_out, const float* w_in,
+                           const float* gamma, void* out, int out_dtype, const int* rows, long long n, int S, int dim,
+                           float eps, dsb200_stream_t stream);
+
 /* ---- csrc/ragged/latent_ops.cu */
 /* out[t, :] = table[ids[t], :] + sinusoid(tok_pos[t]): entry 2i = sin(p f_i), entry 2i + 1 = cos(p f_i); `freq` holds the
  * ceil(dim / 2) frequencies as doubles on the device, or is null for no position vector (tok_pos is then unused).
@@ -456,6 +471,9 @@ int dsb200_clamped_swish_gate(const void* gu, void* out, long long rows, int F, 
 int dsb200_clamped_swish_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, int row_col, void* out,
                                    long long out_ld, long long rows, int F, float alpha, float limit, float shift,
                                    int dtype, dsb200_stream_t stream);
+/* out[r, c] = gelu(gu[r, gate_col0 + c]) * gu[r, up_col0 + c] (tanh form of gelu) for c < F; gu [rows, ld], out [rows, out_ld]; dtype 0 = bf16, 1 = fp32. */
+int dsb200_gelu_gate_cols(const void* gu, long long ld, int gate_col0, int up_col0, void* out, long long out_ld,
+                          long long rows, int F, int dtype, dsb200_stream_t stream);
 /* x[r, c] = cap * tanh(x[r, c] / cap) over fp32 [rows, cols] with row stride ld */
 int dsb200_softcap(float* x, long long ld, long long rows, int cols, float cap, dsb200_stream_t stream);
 /* Router: scores = softmax over the E logits of a token (bias[e], when given, joins the logits first), or (sigmoid_scores) the sigmoid of every
@@ -617,39 +635,45 @@ int dsb200_sink_attention(const void* q, long long q_ld, const void* k_cache, lo
                           dsb200_stream_t stream);
 /* `sink_attention` with learned sinks, a distance term, a mask by parts and free strides:
  *   sink_logit [H] (or null): exp(sink_logit[h]) joins head h's denominator;   r1, r2 [H] (or both null): s_j -= r1[h] ln(1 + r2[h] (pos - j));
+ *   r1 alone: s_j -= r1[h] (pos - j);
  *   part > 0: only the keys of the query's own part of `part` positions (counted from position 0 of the sequence) are visible; window > 0: only
  *   the keys with pos - j < window;
  *   q[t * q_ld + h * q_head_stride + c], out[t * out_ld + h * out_head_stride + c]; a cached key / value head starts every k_row / v_row
- *   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start). */
+ *   elements of its token's row (one plane may serve as keys and as values: pass it twice, with d and dv entries read from a head's start);
+ *   q_group >= H / G: query head h lies in slot (h / (H / G)) q_group + h % (H / G) of its row;  gate (null, or [T, gate_ld] in the activation
+ *   dtype, entry c of head h at h * dv + c): the output times the sigmoid of it. */
 int dsb200_sink_attention_ex(const void* q, long long q_ld, long long q_head_stride, const void* k_cache,
                              long long k_block_stride, int k_row, const void* v_cache, long long v_block_stride, int v_row,
                              const int* tok_seq, const int* tok_pos, const int* block_table, int bt_stride, int block_size,
                              void* out, long long out_ld, long long out_head_stride, int n_tokens, int H, int G, int d,
                              int dv, float scale, float cap, float sink, const float* sink_logit, const float* r1,
-                             const float* r2, int part, int window, int dtype, dsb200_stream_t stream);
+                             const float* r2, int part, int window, int q_group, const void* gate, long long gate_ld,
+                             int dtype, dsb200_stream_t stream);
 /* Low-rank attention with one rotated key part shared by the heads.  proj [T, ld] (dtype 0 = bf16, 1 = fp32) holds per token the H query heads
  * (d plain entries, then dr entries to rotate) from q_col0 and the low-rank row (R entries, then dr entries to rotate) from kv_col0.  The
- * query heads' rotated parts are rotated IN PLACE (first rot_dims of the dr entries; entry i pairs with entry i + rot_dims / 2; angle =
- * pos * freq[i], freq: rot_dims / 2 doubles on the device); the first R entries of the low-rank row are RMS-normed with wkv [R] and, with the
+ * query heads' rotated parts are rotated IN PLACE (first rot_dims of the dr entries; entry i pairs with entry i + rot_dims / 2, or -- interleaved --
+ * entry 2i with entry 2i + 1; angle = pos * freq[i], freq: rot_dims / 2 doubles on the device); the first R entries of the low-rank row are RMS-normed with wkv [R] and, with the
  * rotated last dr entries behind them, written to the token's row of cache [blocks, block_size, row_w] (zeros from R + dr on). */
 int dsb200_latent_rotary_append(void* proj, long long ld, int q_col0, int kv_col0, const float* wkv, const double* freq,
                                 const int* tok_seq, const int* tok_pos, const int* block_table, int bt_stride,
                                 int block_size, void* cache, int row_w, int n_tokens, int H, int d, int dr, int R,
-                                int rot_dims, float eps, int dtype, dsb200_stream_t stream);
+                                int rot_dims, float eps, int interleaved, int dtype, dsb200_stream_t stream);
 /* Attention inputs behind a short causal convolution.  proj [T, ld] holds from col0 on the query heads [H d], the key heads [G d] and the value
  * heads [G dv] of every token; bias (fp32, that many entries, or null) is added to every row before the convolution with conv_w (fp32
  * [taps, channels]: y_t = sum_j w[j, :] u_(t - taps + 1 + j), zeros before the sequence's start).  state [slots, taps - 1, channels]: the last
  * rows of the sequence's earlier steps, WITHOUT the bias (update it afterwards with dsb200_conv_state_update).  Query / key heads: RMS norm over
  * d with wq / wk [d] shared by the heads -> q_out [T, q_ld] (head h at h * q_row) / the key plane.  Value heads: v_own (null, or [T, G dv])
  * receives the convolved values; with v_other ([T, G dv]) and mix (one float on the device) the cached value is (1 - mix) v + mix v_other.
- * Heads are padded with zeros to q_row / k_row / v_row entries. */
+ * Heads are padded with zeros to q_row / k_row / v_row entries.  wq / wk null: the norms have no weight.  q_group >= H / G: query head h goes to
+ * slot (h / (H / G)) q_group + h % (H / G) of its row, slots without a head are zeros.  has_kv = 0: there are only queries (channels [H d]). */
 int dsb200_conv_head_norm_append(const void* proj, long long ld, int col0, const float* bias, const float* conv_w,
                                  const float* wq, const float* wk, const void* state, const int* seq_desc,
                                  const int* tok_seq, const int* tok_pos, const int* block_table, int bt_stride,
                                  int block_size, void* k_cache, long long k_block_stride, void* v_cache,
                                  long long v_block_stride, void* q_out, long long q_ld, const void* v_other,
                                  const float* mix, void* v_own, int n_tokens, int H, int G, int d, int dv, int taps,
-                                 float eps, int q_row, int k_row, int v_row, int dtype, dsb200_stream_t stream);
+                                 float eps, int q_row, int k_row, int v_row, int q_group, int has_kv, int dtype,
+                                 dsb200_stream_t stream);
 
 /* ---- csrc/ragged/ssd_chunk.cu */
 /* The recurrence of dsb200_ssd_scan in its chunked form, for the sequences that bring at least min_new tokens (the others are left to
