@@ -45,21 +45,22 @@ def linear_slopes(H):
 
 
 def sees_window(i, j, size):
-    return j <= i and (size == 0 or i - j < size)
+    return (j <= i) & (i - j < size) if size else j <= i
 
 
 def sees_part(i, j, size):
-    return j <= i and (size == 0 or i // size == j // size)
+    return (j <= i) & (i // size == j // size) if size else j <= i
 
 
 def attend(q, k, v, scale, sees, pos0=0, slopes=None):
-    """q [T, H, d] at positions pos0 ..; k [N, G, d], v [N, G, dv] at positions 0 .. N - 1; sees(i, j): whether query i sees key j;
+    """q [T, H, d] at positions pos0 ..; k [N, G, d], v [N, G, dv] at positions 0 .. N - 1; sees(i, j): whether query i sees key j (tensors of
+    positions);
     slopes [H]: what a score loses per position of distance.  Softmax over what a query sees -> [T, H, dv]."""
     T, H, _ = q.shape
     N, G, _ = k.shape
     per = H // G
     i, j = torch.arange(pos0, pos0 + T)[:, None], torch.arange(N)[None, :]
-    seen = torch.tensor([[bool(sees(int(a), int(b))) for b in range(N)] for a in range(pos0, pos0 + T)])
+    seen = sees(i, j)
     out = torch.zeros(T, H, v.shape[2], dtype=F64)
     for h in range(H):
         s = (q[:, h] @ k[:, h // per].T) * scale
@@ -176,3 +177,106 @@ def forward(config, weights, tokens, carry=None, hook=None):
     logits = linear(rms(X.sum(0), eps) * weights["final.norm"].to(F64), weights, "head")
     cap = float(config.get("logit_softcap", 0.0))
     return (cap * torch.tanh(logits / cap) if cap else logits), {"pos": pos0 + len(tokens), "layers": new}
+
+
+# ------------------------------------------------------------------------------------------------ small models for the tests
+def attention_layer(heads, kv_heads, dim, vdim, chunk, scale=None, conv=3, ff=0, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale if scale is not None else dim ** -0.5}
+    if conv:
+        m["conv"] = conv
+    if chunk:
+        m["mask"] = {"size": chunk}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def latent_layer(heads, dim, rot_dim, vdim, kv_rank, window, scale=None, base=10000.0, ff=0):
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "scale": scale if scale is not None else (dim + rot_dim) ** -0.5,
+         "rot": {"dims": rot_dim, "base": base}}
+    if window:
+        m["mask"] = {"size": window}
+    return {"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def make_config(layers, vocab=64, width=32, eps=1e-5, streams=3, softcap=9.0):
+    return {"architecture": "Ritalorn", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width, "streams": streams, "logit_softcap": softcap}
+
+
+def random_weights(cfg, seed=0):
+    """bf16 tensors under the family's names.  Projections ~ N(0, 1 / fan_in) so that activations stay O(1); mixing matrices that are neither
+    symmetric nor close to the identity; layer scales and stream weights that differ from entry to entry."""
+    g = torch.Generator().manual_seed(seed)
+    D, S = cfg["width"], cfg["streams"]
+
+    def lin(o, i, gain=1.0):
+        return (torch.randn(o, i, generator=g) * gain * i ** -0.5).bfloat16()
+
+    def vec(n, mean=0.0, std=0.2):
+        return (mean + std * torch.randn(n, generator=g)).bfloat16()
+
+    w = {"embed": torch.randn(cfg["vocab"], D, generator=g).bfloat16(), "head": lin(cfg["vocab"], D, 3.0), "final.norm": vec(D, 1.0)}
+
+    def sublayer(p, q):
+        w.update({p + f"norm{q}": vec(D, 1.0), p + f"ls{q}": vec(D, 0.7, 0.3), p + f"hc{q}.in": vec(S, 1.0 / S, 0.4), p + f"hc{q}.out": vec(S, 1.0, 0.4),
+                  p + f"hc{q}.mix": (0.8 * torch.eye(S) + 0.3 * torch.randn(S, S, generator=g)).bfloat16()})
+
+    for i, L in enumerate(cfg["layers"]):
+        m, p, a = L["mixer"], f"l{i}.", f"l{i}.mix."
+        sublayer(p, 1)
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if L["type"] == "attention":
+            G = m["kv_heads"]
+            for name, n in (("q", H * d), ("k", G * d), ("v", G * dv)) if m.get("kv_from") is None else (("q", H * d), ):
+                w.update({a + name: lin(n, D), a + name + ".b": vec(n, 0.0, 0.4)})
+                if m.get("conv"):
+                    w[a + name + ".conv"] = vec((n, m["conv"]), 0.0, 0.8)
+            w.update({a + "g": lin(H * dv, D, 2.0), a + "o": lin(D, H * dv, 2.0), a + "o.b": vec(D)})
+        else:
+            dr, R = m["rot_dim"], m["kv_rank"]
+            w.update({a + "q": lin(H * (d + dr), D, 1.5), a + "dkv": lin(R + dr, D, 1.5), a + "dkv.norm": vec(R, 1.0), a + "uk": lin(H * d, R, 1.5),
+                      a + "uv": lin(H * dv, R), a + "o": lin(D, H * dv, 2.0)})
+        if L["mlp"] is not None:
+            ff = L["mlp"]["ff"]
+            sublayer(p, 2)
+            w.update({p + "mlp.gate": lin(ff, D, 1.5), p + "mlp.up": lin(ff, D, 1.5), p + "mlp.down": lin(D, ff)})
+    return w
+
+
+def run(cfg, w, tokens, collect_layers=False):
+    """Logits of every position of one sequence (float64 [T, vocab]); with collect_layers also the sum of the streams after every layer."""
+    res = []
+    logits, _ = forward(cfg, w, tokens, hook=(lambda i, x: res.append(x.clone())) if collect_layers else None)
+    return (logits, res) if collect_layers else logits
+
+
+def greedy(cfg, w, prompt, n_new):
+    """Greedy continuation, recomputing the whole sequence for every new token."""
+    toks, out = list(prompt), []
+    for _ in range(n_new):
+        nxt = int(run(cfg, w, toks)[-1].argmax())
+        out.append(nxt)
+        toks.append(nxt)
+    return out
+
+
+def write_model(folder, cfg, w):
+    """config.json + model.safetensors (8-byte little-endian header length, JSON header, raw little-endian data) -> folder."""
+    import json
+    import os
+    import struct
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as fh:
+        json.dump(cfg, fh)
+    names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.int32: "I32"}
+    header, blobs, at = {}, [], 0
+    for k, t in w.items():
+        raw = t.contiguous().reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        header[k] = {"dtype": names[t.dtype], "shape": list(t.shape), "data_offsets": [at, at + len(raw)]}
+        blobs.append(raw)
+        at += len(raw)
+    hj = json.dumps(header).encode()
+    hj += b" " * (-len(hj) % 8)
+    with open(os.path.join(folder, "model.safetensors"), "wb") as fh:
+        fh.write(struct.pack("<Q", len(hj)) + hj + b"".join(blobs))
+    return folder
