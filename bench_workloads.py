@@ -1474,5 +1474,283 @@ def run_gepolix(args):
           flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------------------- Ritalorn
+RITALORN_SIZES = {  # width, layers, attention heads, head_dim, kv heads, ff, streams, vocab
+    "s": (2048, 4, 16, 128, 4, 5632, 2, 32000),
+    "m": (4096, 4, 32, 128, 8, 11264, 2, 32000),
+}
+RITALORN_ROT, RITALORN_TAPS, RITALORN_CHUNK = 32, 4, 1024  # rotated entries of the latent rows; convolution taps; chunk and window length
+
+
+def _ritalorn_layout(L):
+    """Kinds of the layers: three attention layers, of which the second reads the first one's cache, and one latent-attention layer, in turn."""
+    return [("attention", "reader", "latent", "attention")[i % 4] for i in range(L)]
+
+
+def _ritalorn_state(torch, dev, W, L, H, d, hkv, ff, S, V):
+    """'attention' (H:hkv heads of d behind 4 taps, chunks of 1024, output gate), one of the same with queries only, 'latent_attention' (H heads of
+    d - 32 plain + 32 rotated entries, values of d, a cached row of d values, window 1024); every layer with a dense feed-forward of ff."""
+    att = {"heads": H, "kv_heads": hkv, "dim": d, "vdim": d, "conv": RITALORN_TAPS, "mask": {"size": RITALORN_CHUNK}, "scale": d ** -0.5}
+    rot = RITALORN_ROT
+    lat = {"heads": H, "dim": d - rot, "rot_dim": rot, "vdim": d, "kv_rank": d - rot, "scale": d ** -0.5, "rot": {"base": 1e6, "dims": rot},
+           "mask": {"size": RITALORN_CHUNK}}
+    layers, owner = [], 0
+    for i, kind in enumerate(_ritalorn_layout(L)):
+        if kind == "attention":
+            owner = i
+        mixer = lat if kind == "latent" else (att if kind == "attention" else dict(att, kv_from=owner))
+        layers.append({"type": "latent_attention" if kind == "latent" else "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+    cfg = {"architecture": "Ritalorn", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "streams": S, "logit_softcap": 30.0, "layers": layers}
+
+    def r(*shape, std=0.02, mean=0.0):
+        return torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(mean, std)
+
+    sd = {"embed": r(V, W, std=1.0), "final.norm": r(W, mean=1.0), "head": r(V, W)}
+    for i, kind in enumerate(_ritalorn_layout(L)):
+        p, a = f"l{i}.", f"l{i}.mix."
+        for q in (1, 2):
+            sd.update({p + f"norm{q}": r(W, mean=1.0), p + f"ls{q}": r(W, mean=0.5), p + f"hc{q}.in": r(S, mean=1.0 / S), p + f"hc{q}.out": r(S, mean=1.0),
+                       p + f"hc{q}.mix": torch.eye(S, device=dev, dtype=torch.bfloat16)})
+        sd.update({p + "mlp.gate": r(ff, W), p + "mlp.up": r(ff, W), p + "mlp.down": r(W, ff)})
+        if kind == "latent":
+            sd.update({a + "q": r(H * d, W), a + "dkv": r(d, W), a + "dkv.norm": r(d - rot, mean=1.0), a + "uk": r(H * (d - rot), d - rot, std=0.1),
+                       a + "uv": r(H * d, d - rot, std=0.1), a + "o": r(W, H * d)})
+            continue
+        for nm, c in (("q", H * d), ("k", hkv * d), ("v", hkv * d))[:1 if kind == "reader" else 3]:
+            sd.update({a + nm: r(c, W), a + nm + ".b": r(c), a + nm + ".conv": r(c, RITALORN_TAPS, std=0.5)})
+        sd.update({a + "g": r(H * d, W), a + "o": r(W, H * d), a + "o.b": r(W)})
+    return cfg, sd
+
+
+def _midulorn_dense_state(torch, dev, W, L, H, d, hkv, ff, V):
+    """The Midulorn of equal size: its attention layers (distance term, sinks, parts) where Ritalorn has attention layers of either kind, its latent
+    layers where Ritalorn has them, dense feed-forwards with as many parameters (xIELU, hidden 3/2 ff)."""
+    rot, dense = MIDULORN_ROT, {"kind": "dense", "ff": 3 * ff // 2}
+    lat = {"type": "latent_attention", "mixer": {"heads": H, "dim": d - rot, "rot_dim": rot, "vdim": d, "kv_rank": d - rot, "scale": d ** -0.5,
+                                                 "rot": {"base": 1e6, "dims": rot}}, "mlp": dense}
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": hkv, "dim": d, "vdim": d, "conv": MIDULORN_TAPS, "mask": {"size": MIDULORN_PART},
+                                          "scale": d ** -0.5, "v_mix": True}, "mlp": dense}
+    layers = [lat if k == "latent" else att for k in _ritalorn_layout(L)]
+    cfg = {"architecture": "Midulorn", "vocab": V, "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": W ** 0.5}, "postln_alpha": 2.0,
+           "logit_scale": 0.25, "layers": layers}
+
+    def r(*shape, std=0.02, mean=0.0):
+        return torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(mean, std)
+
+    sd = {"embed": r(V, W, std=0.05), "final.norm": r(W, mean=1.0)}
+    for i, Lc in enumerate(layers):
+        p, a = f"l{i}.", f"l{i}.mix."
+        sd.update({p + "norm1": r(W, mean=1.0), p + "norm2": r(W, mean=1.0), p + "mlp.up": r(dense["ff"], W), p + "mlp.down": r(W, dense["ff"]),
+                   p + "mlp.act": r(2, std=0.5), a + "sink": r(H, std=1.0), a + "o": r(W, H * d)})
+        if Lc["type"] == "latent_attention":
+            sd.update({a + "q": r(H * d, W), a + "dkv": r(d, W), a + "dkv.norm": r(d - rot, mean=1.0), a + "uk": r(H * (d - rot), d - rot, std=0.1),
+                       a + "uv": r(H * d, d - rot, std=0.1), a + "g": r(H, W)})
+            continue
+        for nm, c in (("q", H * d), ("k", hkv * d), ("v", hkv * d)):
+            sd.update({a + nm: r(c, W), a + nm + ".b": r(c), a + nm + ".conv": r(c, MIDULORN_TAPS, std=0.5)})
+        sd.update({a + "q.norm": r(d, mean=1.0), a + "k.norm": r(d, mean=1.0), a + "vmix": r(1, mean=0.3, std=0.0).reshape(()), a + "r1": r(H, mean=1.0, std=0.1),
+                   a + "r2": r(H, mean=0.5, std=0.05), a + "o.b": r(W)})
+    return cfg, sd
+
+
+def _llama_dense_state(torch, dev, W, L, H, d, hkv, ff, V):
+    cfg = dict(vocab_size=V, hidden_size=W, intermediate_size=ff, num_hidden_layers=L, num_attention_heads=H, num_key_value_heads=hkv, rms_norm_eps=1e-5,
+               rope_theta=1e6, max_position_embeddings=8192)
+
+    def r(*shape, std=0.02, mean=0.0):
+        return torch.empty(*shape, device=dev, dtype=torch.bfloat16).normal_(mean, std)
+
+    sd = {"model.embed_tokens.weight": r(V, W, std=1.0), "model.norm.weight": r(W, mean=1.0), "lm_head.weight": r(V, W)}
+    for i in range(L):
+        p = f"model.layers.{i}."
+        sd.update({p + "self_attn.q_proj.weight": r(H * d, W), p + "self_attn.k_proj.weight": r(hkv * d, W), p + "self_attn.v_proj.weight": r(hkv * d, W),
+                   p + "self_attn.o_proj.weight": r(W, H * d), p + "mlp.gate_proj.weight": r(ff, W), p + "mlp.up_proj.weight": r(ff, W),
+                   p + "mlp.down_proj.weight": r(W, ff), p + "input_layernorm.weight": r(W, mean=1.0), p + "post_attention_layernorm.weight": r(W, mean=1.0)})
+    return cfg, sd
+
+
+def _ritalorn_kernel_table(torch, peaks, W, H, d, hkv, ff, S, T, ctx, n_dec):
+    """Every kernel of the design beside the like kernel of the closest family (Midulorn; Pudinex for the gate of the feed-forward), isolated, with
+    the fraction of the measured roofline (HBM copy bandwidth for the streaming kernels, cuBLAS bf16 rate for attention prefill)."""
+    from deepspeedsyclsupport_b200.inference.v2 import kernels as K
+    dev = torch.device("cuda")
+    bf = torch.bfloat16
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, ms, like, like_ms, nbytes=None, like_bytes=None, flops=None, like_flops=None):
+        def frac(ms_, b, f):
+            return round(max((b or 0) / hbm, (f or 0) / tf) / (ms_ * 1e-3), 3)
+        rows.append({"kernel": name, "ms": round(ms, 4), "roofline_frac": frac(ms, nbytes, flops), "like": like, "like_ms": round(like_ms, 4),
+                     "like_roofline_frac": frac(like_ms, like_bytes if like_bytes is not None else nbytes, like_flops if like_flops is not None else flops)})
+
+    rot, taps, chunk = RITALORN_ROT, RITALORN_TAPS, RITALORN_CHUNK
+    g32, y = torch.randn(W, device=dev), torch.randn(T, W, device=dev).to(bf)
+    for label, n in (("prefill", T), ("decode", n_dec)):
+        x1, yn = torch.randn(n, W, device=dev), y[:n]
+        ms_like = _event_ms(torch, lambda: K.post_sum_norm(x1, yn, g32, 2.0, 1e-6, bias=g32), 20, flush)
+        for s in sorted({2, 4, S}):
+            X = torch.randn(n, s, W, device=dev)
+            co = (yn, g32, g32, torch.eye(s, device=dev), torch.ones(s, device=dev))
+            w_in = torch.full((s, ), 1.0 / s, device=dev)
+            add(f"stream_mix_norm ({s} streams; bf16 branch + bias + scale in, streams and bf16 norm out), {label}",
+                _event_ms(torch, lambda: K.stream_mix_norm(X, s, co, w_in, g32), 20, flush), f"post_sum_norm (bf16 branch + bias; Midulorn), {label}", ms_like,
+                nbytes=n * W * (8 * s + 4), like_bytes=n * W * 12)
+        gu, act = torch.randn(n, 2 * ff, device=dev).to(bf), torch.empty(n, ff, device=dev, dtype=bf)
+        add(f"gelu_gate_cols, {label}", _event_ms(torch, lambda: K.gelu_gate_cols(gu, 0, ff, ff, act), 20, flush), f"clamped_swish_gate_cols (Pudinex), {label}",
+            _event_ms(torch, lambda: K.clamped_swish_gate_cols(gu, 0, ff, ff, act, 1.0, float("inf"), 0.0), 20, flush), nbytes=n * ff * 6)
+    bs = 128
+    lfreq = torch.tensor([1e6 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=dev)
+    Hp = 1 << (H - 1).bit_length()
+    for label, n_seq, new, seen in (("prefill", max(1, T // 2048), min(T, 2048), ctx), ("decode", n_dec, 1, ctx)):
+        per = -(-(seen + new) // bs)
+        nb = n_seq * per
+        bt = torch.arange(nb, dtype=torch.int32, device=dev).view(n_seq, per)
+        tok_seq = torch.arange(n_seq, dtype=torch.int32, device=dev).repeat_interleave(new)
+        tok_pos = (seen + torch.arange(new, dtype=torch.int32, device=dev)).repeat(n_seq)
+        desc = torch.tensor([[i * new, new, seen, i] for i in range(n_seq)], dtype=torch.int32, device=dev)
+        Tn = n_seq * new
+        dec = label == "decode"
+        C, n = (H + 2 * hkv) * d, H * d
+        kv = torch.randn(nb, 2, bs, hkv, d, device=dev).to(bf)
+        planes = K.cache_planes(kv)
+        proj = torch.randn(Tn, C + n, device=dev).to(bf)  # queries | keys | values | output gate
+        gate = proj[:, C:]
+        qo = torch.empty(Tn, n, device=dev, dtype=bf)
+        nw = torch.randn(d, device=dev)
+        cw, cb, mix = torch.randn(taps, C, device=dev), torch.randn(C, device=dev), torch.full((1, ), 0.3, device=dev)
+        cwq, cbq = cw[:, :n].contiguous(), cb[:n].contiguous()
+        cstate, cstate_q = (torch.zeros(n_seq, taps - 1, c, device=dev, dtype=bf) for c in (C, n))
+        vsrc = torch.randn(Tn, hkv * d, device=dev).to(bf)
+
+        def prep(w, b, st, c, norm=None, kv_=True, **kw):
+            K.conv_head_norm_append(proj, 0, b, w, norm, norm, st, desc, tok_seq, tok_pos, bt, bs, planes[0], planes[1], qo, H, hkv, d, d, taps, 1e-6, kv=kv_, **kw)
+            K.conv_state_update(proj, 0, c, st, 0, desc, n_seq, taps)
+
+        ms_like = _event_ms(torch, lambda: prep(cw, cb, cstate, C, norm=nw, v_other=vsrc, mix=mix), 10, flush)
+        like = f"conv_head_norm_append + conv_state_update (norm weights, mixed values; Midulorn), {label}"
+        add(f"conv_head_norm_append + conv_state_update, {label}", _event_ms(torch, lambda: prep(cw, cb, cstate, C), 10, flush), like, ms_like,
+            nbytes=Tn * C * 4, like_bytes=Tn * (C * 4 + hkv * d * 2))
+        add(f"conv_head_norm_append + conv_state_update, queries only, {label}", _event_ms(torch, lambda: prep(cwq, cbq, cstate_q, n, kv_=False), 10, flush), like,
+            ms_like, nbytes=Tn * n * 4, like_bytes=Tn * (C * 4 + hkv * d * 2))
+        out = torch.empty(Tn, n, device=dev, dtype=bf)
+        sl = torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], device=dev)
+        r1, r2, sk = torch.full((H, ), 1.0, device=dev), torch.full((H, ), 0.5, device=dev), torch.randn(H, device=dev)
+        where = (tok_seq, tok_pos, bt)
+        for part in (1 << 20, chunk):
+            pk = n_seq * sum(min(p % part + 1, p + 1) for p in range(seen, seen + new))
+            kvb = n_seq * min(seen + new, part + new) * hkv * d * 4
+            what = "one chunk" if part > seen + new else f"chunks of {part}"
+            add(f"attention, linear distance term + output gate, {what}, tcgen05, {label} (GQA {H}:{hkv})",
+                _event_ms(torch, lambda: K.paged_flash_sink(qo, kv, *where, out, H, hkv, d, d ** -0.5, 0.0, 0.0, decode=dec, r1=sl, part=part,
+                                                            compact=(H // hkv, d), gate=gate), 10, flush),
+                f"attention, logarithmic distance term + learned sinks, {what}, tcgen05, {label} (Midulorn)",
+                _event_ms(torch, lambda: K.paged_flash_sink(qo, kv, *where, out, H, hkv, d, d ** -0.5, 0.0, 0.0, decode=dec, sink_logit=sk, r1=r1, r2=r2, part=part), 10,
+                          flush),
+                nbytes=kvb + Tn * n * 6, like_bytes=kvb + Tn * n * 4, flops=4.0 * pk * n)
+        lat = torch.randn(Tn, n + d, device=dev).to(bf)
+        lcache = torch.randn(nb, bs, d, device=dev).to(bf)
+        wkv = torch.randn(d - rot, device=dev)
+
+        def append(inter):
+            K.latent_rotary_append(lat, 0, n, wkv, lfreq, tok_seq, tok_pos, bt, lcache, H, d - rot, rot, d - rot, rot, 1e-6, interleaved=inter)
+        add(f"latent_rotary_append, neighbouring pairs, {label}", _event_ms(torch, lambda: append(True), 10, flush), f"latent_rotary_append, halves (Midulorn), {label}",
+            _event_ms(torch, lambda: append(False), 10, flush), nbytes=Tn * (H * rot * 4 + d * 4))
+        qa = torch.randn(Hp, Tn, d, device=dev).to(bf)
+        skp = torch.randn(Hp, device=dev)
+        wk = n_seq * sum(min(p + 1, chunk) for p in range(seen, seen + new))
+        keys = n_seq * new * (seen + (new + 1) / 2)
+        add(f"latent attention, window {chunk}, tcgen05 one-plane, {label} ({Hp} heads)",
+            _event_ms(torch, lambda: K.paged_latent_flash(qa.transpose(0, 1), lcache, *where, d ** -0.5, decode=dec, heads=Hp, window=chunk), 10, flush),
+            f"latent attention with learned sinks, tcgen05 one-plane, {label} (Midulorn; whole context)",
+            _event_ms(torch, lambda: K.paged_latent_flash(qa.transpose(0, 1), lcache, *where, d ** -0.5, decode=dec, heads=Hp, sink_logit=skp), 10, flush),
+            nbytes=n_seq * min(seen + new, chunk + new) * d * 2 + Tn * Hp * d * 4, like_bytes=n_seq * (seen + new) * d * 2 + Tn * Hp * d * 4,
+            flops=4.0 * wk * Hp * d, like_flops=4.0 * keys * Hp * d)
+    return rows
+
+
+def run_ritalorn(args):
+    """Prefill and decode throughput of Ritalorn through the FastGen engine at a few layer sizes, beside a Midulorn (the closest family: convolved
+    attention with a distance term and a mask by parts, low-rank attention) and a Llama of equal size (same width, layers, heads, kv heads,
+    feed-forward parameters, vocabulary), plus the isolated kernels of the design beside their likes."""
+    sys.path.insert(0, ROOT)
+    import torch
+    import deepspeedsyclsupport_b200 as deepspeed
+    from deepspeedsyclsupport_b200 import comm as dist
+    from deepspeedsyclsupport_b200.inference.v2 import RaggedInferenceEngineConfig, build_engine_from_state_dict
+    from deepspeedsyclsupport_b200.ops import native
+    deepspeed.init_distributed()
+    assert dist.get_world_size() == 1, "--workload ritalorn is a one-GPU comparison"
+    dev = torch.device("cuda", torch.cuda.current_device())
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "source": "fallback"}
+    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+        peaks = dict(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json"))), source="measured")
+    n_seqs, prompt, budget = min(args.sequences, 64), 1024, 4096
+    results, clocks, l0 = {}, None, native.launch_count
+    g = torch.Generator().manual_seed(11)
+    for name in (args.model.split(",") if args.model != "7b" else ["s", "m"]):
+        W, L, H, d, hkv, ff, S, V = RITALORN_SIZES[name]
+        max_ctx = -(-(prompt + 4 * (args.steps + args.warmup) * 4 + 64) // 128) * 128
+        ecfg = RaggedInferenceEngineConfig(state_manager={"max_ragged_batch_size": budget, "max_ragged_sequence_count": n_seqs, "max_tracked_sequences": n_seqs,
+                                                          "max_context": max_ctx, "memory_config": {"mode": "allocate", "size": n_seqs * (max_ctx // 128) + 4}})
+        res = {}
+        for fam in ("ritalorn", "midulorn", "llama"):
+            if fam == "ritalorn":
+                cfg, sd = _ritalorn_state(torch, dev, W, L, H, d, hkv, ff, S, V)
+            else:
+                cfg, sd = (_midulorn_dense_state if fam == "midulorn" else _llama_dense_state)(torch, dev, W, L, H, d, hkv, ff, V)
+            eng = build_engine_from_state_dict(fam, cfg, sd, ecfg, dtype=torch.bfloat16)
+            n_params = sum(v.numel() for v in sd.values())
+            del sd
+            prompts = [torch.randint(0, V, (prompt, ), generator=g).pin_memory() for _ in range(n_seqs)]
+            uids = list(range(n_seqs))
+            state = {"live": False, "next": None}
+
+            def prefill():
+                if state["live"]:
+                    for u in uids:
+                        eng.flush(u)
+                per = budget // prompt
+                nxt = torch.zeros(n_seqs, dtype=torch.long)
+                for i in range(0, n_seqs, per):
+                    us = uids[i:i + per]
+                    nxt[i:i + len(us)] = eng.put(us, [prompts[u] for u in us]).argmax(-1).cpu()
+                state["live"], state["next"] = True, nxt
+
+            def decode():
+                nxt = state["next"]
+                for _ in range(4):
+                    nxt = eng.put(uids, [nxt[u:u + 1] for u in uids]).argmax(-1).cpu()
+                state["next"] = nxt
+
+            ms_p, _ = _timed(torch, dist, prefill, args.steps, 3)
+            ms_d, clk = _timed(torch, dist, decode, args.steps, args.warmup)
+            if fam == "ritalorn":
+                clocks = clk
+            res[fam] = {"params_b": round(n_params / 1e9, 3), "prefill_tokens_per_s": round(n_seqs * prompt / ms_p * 1e3, 1), "prefill_ms": round(ms_p, 2),
+                        "decode_tokens_per_s": round(n_seqs * 4 / ms_d * 1e3, 1), "decode_ms_per_step": round(ms_d / 4, 3)}
+            del eng
+            torch.cuda.empty_cache()
+        for other in ("midulorn", "llama"):
+            res["ritalorn_over_" + other] = {"prefill": round(res["ritalorn"]["prefill_tokens_per_s"] / res[other]["prefill_tokens_per_s"], 3),
+                                             "decode": round(res["ritalorn"]["decode_tokens_per_s"] / res[other]["decode_tokens_per_s"], 3)}
+        res["shape"] = {"width": W, "layers": L, "heads": H, "head_dim": d, "kv_heads": hkv, "ff": ff, "streams": S, "rotated": RITALORN_ROT, "taps": RITALORN_TAPS,
+                        "chunk and window": RITALORN_CHUNK}
+        res["kernels"] = _ritalorn_kernel_table(torch, peaks, W, H, d, hkv, ff, S, 4096, 2048, n_seqs)
+        results[name] = res
+    launches = native.launch_count - l0
+    last = results[list(results)[-1]]
+    extra = {"results": results, "peaks": {k: peaks[k] for k in ("hbm_gbs", "bf16_tflops", "source")},
+             "e2e": {"value": last["ritalorn"]["decode_tokens_per_s"], "unit": "generated tokens/s", "h2d_bytes_per_step": n_seqs * 8, "d2h_bytes_per_step": n_seqs * 8},
+             "reference_arm": "none: the reference has no model of this design"}
+    config = {"model": "ritalorn (random weights) beside midulorn and llama of equal size", "sizes": list(results), "sequences": n_seqs, "prompt_len": prompt,
+              "token_budget_per_forward": budget, "decode_steps_per_timed_step": 4, "kv_block": 128,
+              "l2_policy": "engine steps: weights exceed the 126 MB L2, no flush; isolated kernels: 256 MB write before every timed run"}
+    print(json.dumps(_line("generated tokens/sec Ritalorn FastGen ragged decode, 1 GPU (prefill, a Midulorn and a Llama of equal size alongside)",
+                           last["ritalorn"]["decode_tokens_per_s"], "tokens/s", 1, args, last["ritalorn"]["decode_ms_per_step"], config, clocks, launches, extra)),
+          flush=True)
+
+
 WORKLOADS = {"fastgen70b": run_fastgen70b, "mixtral": run_mixtral, "ulysses13b": run_ulysses13b, "linasun": run_linasun, "kulanex": run_kulanex, "pudinex": run_pudinex, "midulorn": run_midulorn,
-             "gepolix": run_gepolix}
+             "gepolix": run_gepolix, "ritalorn": run_ritalorn}
